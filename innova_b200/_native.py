@@ -55,6 +55,16 @@ def lib_dir() -> Path:
     return Path(__file__).resolve().parent / "lib"
 
 
+_subset = None
+
+
+def use_subset(group: str, cuda_sources, host_sources):
+    """If the full libraries are not built, build and load only the named sources (before the first kernel call). A command
+    that serves one kind of model calls this so that a fresh checkout compiles what that model needs and no more."""
+    global _subset
+    _subset = (group, tuple(cuda_sources), tuple(host_sources))
+
+
 def cuda():
     """The CUDA kernel library (built in-tree on first use)."""
     global _cuda
@@ -64,7 +74,10 @@ def cuda():
                 path = lib_dir() / "libinnova_cuda.so"
                 if not path.exists():
                     from . import build
-                    build.build_cuda()
+                    if _subset is None:
+                        build.build_cuda()
+                    else:
+                        path = build.build_subset(_subset[0] + "_cuda", _subset[1])
                 _cuda = _bind(C.CDLL(str(path)), _CUDA_SIGS)
     return _cuda
 
@@ -86,7 +99,10 @@ def host():
                 path = Path(override) if override else lib_dir() / "libinnova_host.so"
                 if not path.exists():
                     from . import build
-                    build.build_host()
+                    if _subset is None or override:
+                        build.build_host()
+                    else:
+                        path = build.build_subset(_subset[0] + "_host", _subset[2], host=True)
                 _host = C.CDLL(str(path))
     return _host
 

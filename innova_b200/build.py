@@ -25,6 +25,8 @@ NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-O3",
 ]
+# Sources whose arithmetic also serves the fp32 models: IEEE division and square root, accurate exponentials.
+PRECISE_SOURCES = {"hyper.cu", "delta_rule.cu", "latent_attn.cu"}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function", "-pthread"]
 
 
@@ -55,9 +57,23 @@ def host_sources():
     return sorted((CSRC / "host").glob("*.cpp"))
 
 
-def build_cuda(force: bool = False, verbose: bool = False) -> Path:
-    out = LIB / "libinnova_cuda.so"
-    srcs = cuda_sources()
+def nvcc_flags(src: Path):
+    return [f for f in NVCC_FLAGS if not (f == "--use_fast_math" and src.name in PRECISE_SOURCES)]
+
+
+def subset_lib(group: str) -> Path:
+    return LIB / f"libinnova_{group}.so"
+
+
+def build_subset(group: str, names, host: bool = False) -> Path:
+    """A library of the named sources only (``csrc/*.cu``, or ``csrc/host/*.cpp`` with ``host``): what a command that runs one
+    family of models compiles in a fresh checkout. It exports the same symbols as the full library."""
+    return build_host(only=set(names), out=subset_lib(group)) if host else build_cuda(only=set(names), out=subset_lib(group))
+
+
+def build_cuda(force: bool = False, verbose: bool = False, only=None, out: Path | None = None) -> Path:
+    out = out or LIB / "libinnova_cuda.so"
+    srcs = [s for s in cuda_sources() if only is None or s.name in only]
     headers = list(CSRC.glob("*.cuh")) + list(CSRC.glob("*.h"))
     nvcc = _nvcc()
     if nvcc is None:
@@ -69,7 +85,7 @@ def build_cuda(force: bool = False, verbose: bool = False) -> Path:
     for s in srcs:
         o = OBJ / (s.stem + ".o")
         if force or _newer([s] + headers, o):
-            cmd = [nvcc, *NVCC_FLAGS, "-I", str(CSRC), "-c", str(s), "-o", str(o)]
+            cmd = [nvcc, *nvcc_flags(s), "-I", str(CSRC), "-c", str(s), "-o", str(o)]
             if verbose:
                 cmd.insert(1, "-Xptxas=-v")
             jobs.append(cmd)
@@ -84,9 +100,9 @@ def build_cuda(force: bool = False, verbose: bool = False) -> Path:
     return out
 
 
-def build_host(force: bool = False) -> Path:
-    out = LIB / "libinnova_host.so"
-    srcs = host_sources()
+def build_host(force: bool = False, only=None, out: Path | None = None) -> Path:
+    out = out or LIB / "libinnova_host.so"
+    srcs = [s for s in host_sources() if only is None or s.name in only]
     if not srcs:
         return out
     headers = list((CSRC / "host").glob("*.h"))

@@ -32,6 +32,7 @@ struct FlashFwdParams {
   float scale;
   int causal;
   int window;  // > 0 (causal only): a query sees the `window` most recent keys, its own position included
+  const int* cu;  // packed batch: sequence b is rows [cu[b], cu[b + 1]) of the token-major buffers; null: B sequences of S rows
   int* status;
 };
 
@@ -82,12 +83,16 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int nqb = (p.S + FA_BM - 1) / FA_BM;
-  const int q_blk = nqb - 1 - blockIdx.x;
   const int h = blockIdx.y, b = blockIdx.z;
+  const int row_base = p.cu ? p.cu[b] : 0;      // first row of the sequence in its tensor-map slice
+  const int S = p.cu ? p.cu[b + 1] - row_base : p.S;
+  const int bz = p.cu ? 0 : b;
+  const int nqb = (S + FA_BM - 1) / FA_BM;
+  const int q_blk = nqb - 1 - (int)blockIdx.x;
+  if (q_blk < 0) return;                        // packed batches: the grid covers the longest sequence
   const int hk = h / (p.H / p.Hkv);
   const int q0 = q_blk * FA_BM;
-  const int nkb_all = (p.S + FA_BN - 1) / FA_BN;
+  const int nkb_all = (S + FA_BN - 1) / FA_BN;
   // key blocks visited: [jlo, jlo + nkb). A sliding window skips the blocks that lie wholly before the first query's window.
   const int jlo = (p.causal && p.window > 0) ? max(0, q0 - p.window + 1) / FA_BN : 0;
   const int nkb = (p.causal ? min(nkb_all, q_blk + 1) : nkb_all) - jlo;
@@ -123,7 +128,7 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     if (lane == 0) {
       mbar_expect_tx(q_full, L::TILE);
 #pragma unroll
-      for (int a = 0; a < ND; ++a) tma_load_3d(sQ + a * 16384, &tmap_q, q_full, h * D + a * 64, q0, b);
+      for (int a = 0; a < ND; ++a) tma_load_3d(sQ + a * 16384, &tmap_q, q_full, h * D + a * 64, row_base + q0, bz);
       for (int n = 0; n < 2 * nkb; ++n) {
         const int slot = n % SLOTS;
         const uint32_t ph = (n / SLOTS) & 1;
@@ -132,7 +137,7 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         const int j = jlo + (n >> 1);
         const CUtensorMap* tm = (n & 1) ? &tmap_v : &tmap_k;
 #pragma unroll
-        for (int a = 0; a < ND; ++a) tma_load_3d(sKV + slot * L::TILE + a * 16384, tm, &kv_full[slot], hk * D + a * 64, j * FA_BN, b);
+        for (int a = 0; a < ND; ++a) tma_load_3d(sKV + slot * L::TILE + a * 16384, tm, &kv_full[slot], hk * D + a * 64, row_base + j * FA_BN, bz);
       }
     }
   } else if (warp == 1) {
@@ -188,8 +193,8 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       tc_fence_after();
       const int k0 = (jlo + j) * FA_BN;
       const bool windowed = p.causal && p.window > 0;
-      const bool need_mask = (p.causal && k0 + FA_BN - 1 > q0) || (k0 + FA_BN > p.S) || (windowed && k0 <= q0 + FA_BM - 1 - p.window);
-      const int kmax = p.causal ? min(row, p.S - 1) : p.S - 1;
+      const bool need_mask = (p.causal && k0 + FA_BN - 1 > q0) || (k0 + FA_BN > S) || (windowed && k0 <= q0 + FA_BM - 1 - p.window);
+      const int kmax = p.causal ? min(row, S - 1) : S - 1;
       const int kmin = windowed ? row - p.window + 1 : 0;
       uint32_t sr[128];
       tmem_ld_32x32(t_lane, sr);
@@ -259,13 +264,13 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     if (ok) {
       tc_fence_after();
       const float inv_l = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* dst = p.out + ((size_t)b * p.S + row) * p.ld_o + h * D;
+      __nv_bfloat16* dst = p.out + ((p.cu ? (size_t)row_base : (size_t)b * S) + row) * p.ld_o + h * D;
 #pragma unroll 1
       for (int cc = 0; cc < D / 32; ++cc) {
         uint32_t rr[32];
         tmem_ld_32x32(t_lane + O_COL + cc * 32, rr);
         tmem_ld_wait();
-        if (row < p.S) {
+        if (row < S) {
 #pragma unroll
           for (int g = 0; g < 4; ++g) {
             uint4 o;
@@ -277,7 +282,7 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
           }
         }
       }
-      if (p.lse && row < p.S) p.lse[((size_t)b * p.H + h) * p.S + row] = m_used * c + log2f(l);
+      if (p.lse && row < S) p.lse[((size_t)b * p.H + h) * S + row] = m_used * c + log2f(l);
       tc_fence_before();
     }
   }
@@ -340,23 +345,22 @@ int make_tmap_tokens_f32(CUtensorMap* out, const void* ptr, int cols, int S, int
 
 using namespace inv;
 
-// q/k/v: token-major bf16 [B*S, ld*]; q has H heads, k and v have Hkv heads of `head_dim` columns.
-// out: [B*S, ld_o] bf16; lse: [B, H, S] fp32 (may be null).
-extern "C" int inv_flash_attn_fwd(const void* q, const void* k, const void* v, void* out, float* lse, int B, int S, int H, int Hkv,
-                                  int head_dim, int ld_q, int ld_k, int ld_v, int ld_o, float scale, int causal, int window, int* status,
-                                  void* stream) {
+static int flash_fwd_launch(const void* q, const void* k, const void* v, void* out, float* lse, const int* cu, int n_seq, int max_len, int map_b,
+                            int map_s, int H, int Hkv, int head_dim, int ld_q, int ld_k, int ld_v, int ld_o, float scale, int causal, int window,
+                            int* status, void* stream) {
   if ((head_dim != 64 && head_dim != 128) || H % Hkv || (ld_q % 8) || (ld_k % 8) || (ld_v % 8) || (ld_o % 8)) return -ERR_BAD_ARG;
   if (window < 0 || (window > 0 && !causal)) return -ERR_BAD_ARG;  // the sliding window is defined for causal attention
-  if (B <= 0 || S <= 0) return 0;
+  if (n_seq <= 0 || max_len <= 0) return 0;
   CUtensorMap tq, tk, tv;
   int rc;
-  if ((rc = make_tmap_tokens_bf16(&tq, q, H * head_dim, S, B, ld_q, FA_BM))) return rc;
-  if ((rc = make_tmap_tokens_bf16(&tk, k, Hkv * head_dim, S, B, ld_k, FA_BN))) return rc;
-  if ((rc = make_tmap_tokens_bf16(&tv, v, Hkv * head_dim, S, B, ld_v, FA_BN))) return rc;
+  if ((rc = make_tmap_tokens_bf16(&tq, q, H * head_dim, map_s, map_b, ld_q, FA_BM))) return rc;
+  if ((rc = make_tmap_tokens_bf16(&tk, k, Hkv * head_dim, map_s, map_b, ld_k, FA_BN))) return rc;
+  if ((rc = make_tmap_tokens_bf16(&tv, v, Hkv * head_dim, map_s, map_b, ld_v, FA_BN))) return rc;
   FlashFwdParams p;
   p.out = (__nv_bfloat16*)out; p.ld_o = ld_o; p.lse = lse;
-  p.B = B; p.S = S; p.H = H; p.Hkv = Hkv; p.scale = scale; p.causal = causal; p.window = 0; p.status = status;
-  dim3 grid((S + FA_BM - 1) / FA_BM, H, B);
+  p.B = n_seq; p.S = max_len; p.H = H; p.Hkv = Hkv; p.scale = scale; p.causal = causal ? 1 : 0; p.status = status; p.cu = cu;
+  p.window = window >= max_len ? 0 : window;
+  dim3 grid((max_len + FA_BM - 1) / FA_BM, H, n_seq);
   cudaStream_t st = (cudaStream_t)stream;
   static bool configured = false;
   if (!configured) {
@@ -364,10 +368,25 @@ extern "C" int inv_flash_attn_fwd(const void* q, const void* k, const void* v, v
     cudaFuncSetAttribute(flash_fwd3_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, Fwd3Smem<2>::TOTAL);
     configured = true;
   }
-  p.causal = causal ? 1 : 0;
-  p.window = window >= S ? 0 : window;
   if (head_dim == 64) flash_fwd3_kernel<1><<<grid, FA_THREADS, Fwd3Smem<1>::TOTAL, st>>>(tq, tk, tv, p);
   else flash_fwd3_kernel<2><<<grid, FA_THREADS, Fwd3Smem<2>::TOTAL, st>>>(tq, tk, tv, p);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
+}
+
+// q/k/v: token-major bf16 [B*S, ld*]; q has H heads, k and v have Hkv heads of `head_dim` columns.
+// out: [B*S, ld_o] bf16; lse: [B, H, S] fp32 (may be null).
+extern "C" int inv_flash_attn_fwd(const void* q, const void* k, const void* v, void* out, float* lse, int B, int S, int H, int Hkv,
+                                  int head_dim, int ld_q, int ld_k, int ld_v, int ld_o, float scale, int causal, int window, int* status,
+                                  void* stream) {
+  return flash_fwd_launch(q, k, v, out, lse, nullptr, B, S, B, S, H, Hkv, head_dim, ld_q, ld_k, ld_v, ld_o, scale, causal, window, status, stream);
+}
+
+// Packed sequences: rows [cu[i], cu[i + 1]) of [T, ld*] are sequence i (cu: n_seq + 1 device ints, cu[n_seq] = T, none longer
+// than max_len). Causal. A tile that reaches past its sequence reads the next one's rows, which the mask removes.
+extern "C" int inv_flash_attn_packed(const void* q, const void* k, const void* v, void* out, const int* cu, int n_seq, int T, int max_len, int H,
+                                     int Hkv, int head_dim, int ld_q, int ld_k, int ld_v, int ld_o, float scale, int window, int* status,
+                                     void* stream) {
+  if (T <= 0) return 0;
+  return flash_fwd_launch(q, k, v, out, nullptr, cu, n_seq, max_len, 1, T, H, Hkv, head_dim, ld_q, ld_k, ld_v, ld_o, scale, 1, window, status, stream);
 }

@@ -11,6 +11,7 @@ reference-written one (no tail: the extras are inferred from the tensor names).
 from __future__ import annotations
 
 import json
+import os
 from typing import Callable, Dict, Optional, Union
 
 import torch
@@ -22,14 +23,20 @@ _TAIL_TAG = b"\0INVCFG1"
 _KEEP_FP32 = ("norm.weight", "norm.bias", ".bias")
 
 
-def config_blob(cfg: TransformerConfig) -> bytes:
+def config_blob(cfg) -> bytes:
+    if not isinstance(cfg, TransformerConfig):     # a registered architecture: the struct carries what it has room for
+        head = TransformerConfig(vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size, num_layers=cfg.num_layers, max_seq_len=cfg.max_seq_len)
+        return head.pack_reference_struct() + _TAIL_TAG + json.dumps(cfg.to_dict()).encode()
     return cfg.pack_reference_struct() + _TAIL_TAG + json.dumps(cfg.to_dict()).encode()
 
 
 def parse_config(blob: bytes, tensor_names=()) -> Optional[TransformerConfig]:
     if len(blob) >= 88 and _TAIL_TAG in blob[88:]:
-        tail = blob[blob.index(_TAIL_TAG, 88) + len(_TAIL_TAG):]
-        return TransformerConfig(**json.loads(tail.decode()))
+        tail = json.loads(blob[blob.index(_TAIL_TAG, 88) + len(_TAIL_TAG):].decode())
+        if "architecture" in tail:
+            from ..models.registry import model_class
+            return model_class(tail).config_class.from_dict(tail)
+        return TransformerConfig(**tail)
     if len(blob) >= 88:
         cfg = TransformerConfig.unpack_reference_struct(blob)
     elif len(blob) >= 65:
@@ -81,14 +88,37 @@ def load_state(path: str) -> Dict[str, torch.Tensor]:
         return {n: r.read_tensor(n) for n in r.tensor_names()}
 
 
+def read_config_dir(path: str) -> dict:
+    with open(os.path.join(path, "config.json")) as f:
+        return json.load(f)
+
+
+def load_model_dir(path: str, dtype=torch.bfloat16, device="cpu"):
+    """A directory with ``config.json`` (its ``architecture`` names a registered model) and ``model.safetensors``."""
+    from ..models.registry import model_class
+    from .importers import TensorFile
+    config = read_config_dir(path)
+    with TensorFile(os.path.join(path, "model.safetensors"), "safetensors") as f:
+        tensors = dict(f.items())
+    return model_class(config).from_tensors(config, tensors, dtype, device)
+
+
 def load_model(path: str, dtype=torch.float32, device="cpu", ref_layout: bool = False, config: Optional[TransformerConfig] = None):
-    """-> DenseModel (or MoEModel when the file holds experts) with the file's weights."""
+    """-> DenseModel (or MoEModel when the file holds experts) with the file's weights, or a model of a registered architecture
+    when the header names one or ``path`` is a directory with ``config.json``."""
+    if os.path.isdir(path):
+        return load_model_dir(path, dtype, device)
     with oil.OILReader(path) as r:
         names = r.tensor_names()
         cfg = config or parse_config(r.config, names)
         if cfg is None:
             raise ValueError(f"{path}: no usable config in the header; pass config=")
         tensors = {n: r.read_tensor(n) for n in names}
+    if not isinstance(cfg, TransformerConfig):
+        from ..models.registry import model_class
+        shapes = cfg.tensor_shapes()
+        conf = cfg.to_dict()
+        return model_class(conf).from_tensors(conf, {n: t.view(shapes[n]) for n, t in tensors.items() if n in shapes}, dtype, device)
     if any(".moe." in n for n in names):
         from ..models.moe import MoEModel
         model = MoEModel(cfg, dtype=dtype)

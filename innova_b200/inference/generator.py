@@ -36,23 +36,34 @@ class GenerationStats:
 
 
 class Generator:
-    def __init__(self, model, tokenizer=None, kv_format: str = "oil4", max_batch: int = 1, max_seq: Optional[int] = None, linear_fn=None):
+    def __init__(self, model, tokenizer=None, kv_format: str = "oil4", max_batch: int = 1, max_seq: Optional[int] = None, linear_fn=None,
+                 num_pages: Optional[int] = None):
         self.model = model.eval()
         self.cfg = model.cfg
         self.tok = tokenizer
         self.device = next(model.parameters()).device
         self.max_seq = max_seq or self.cfg.max_seq_len
+        self.stats = GenerationStats()
+        # models of the registry bring their own cache and step function; the rest run the dense decoder's step below
+        self.stepped = hasattr(model, "make_cache")
+        if self.stepped:
+            self.cache = model.make_cache(max_batch, self.max_seq, self.device, num_pages)
+            self._graphs, self._warm, self.use_graphs = {}, {}, self.device.type == "cuda"
+            return
         if self.device.type != "cuda" and kv_format == "oil4" and self.cfg.head_dim % 32:
             kv_format = "bf16"
         self.cache = PagedKVCache(self.cfg.num_layers, self.cfg.kv_heads, self.cfg.head_dim, max_batch, self.max_seq, self.device, kv_format)
         self.linear = linear_fn or (lambda x, lin: ops.linear(x, lin.weight, lin.bias))
-        self.stats = GenerationStats()
 
     # ------------------------------------------------------------------ one forward over new tokens
     @torch.no_grad()
     def _forward(self, ids: torch.Tensor, start: List[int], all_logits: bool = False, slots: Optional[List[int]] = None) -> torch.Tensor:
         """ids [B, S_new]; sequences 0..B-1 continue at positions start[b]. Returns logits [B, vocab] of the
         last new token, or [B, S_new, vocab] with ``all_logits`` (speculative verification)."""
+        if self.stepped:
+            B, S = ids.shape
+            out = self.step(ids.tolist(), start, list(range(B)) if slots is None else slots, want=range(B * S) if all_logits else None)
+            return out.view(B, S, -1) if all_logits else out
         m, cfg, cache = self.model, self.cfg, self.cache
         B, S = ids.shape
         H, Hkv, D = cfg.num_heads, cfg.kv_heads, cfg.head_dim
@@ -108,6 +119,47 @@ class Generator:
         logits = ops.linear(last, m.lm_head.weight)
         return logits[..., : cfg.vocab_size]
 
+    # ------------------------------------------------------------------ packed step (models of the registry)
+    GRAPH_WARMUP, MAX_GRAPHS = 2, 16
+
+    @torch.no_grad()
+    def step(self, tokens: Sequence[Sequence[int]], start: Sequence[int], rows: Sequence[int], want: Optional[Sequence[int]] = None):
+        """One step of a batch of unequal requests: ``tokens[i]`` (any number) continue cache row ``rows[i]`` at ``start[i]``.
+        Returns the logits of the packed positions ``want`` (default: the last of each request), None if ``want`` is empty.
+        Steps of one token per request are captured in a CUDA graph once their batch size has come up a few times."""
+        from .state_cache import StepBatch
+        if not self.stepped:
+            raise NotImplementedError("packed steps are for models with their own step function")
+        ends = [s + len(t) for s, t in zip(start, tokens)]
+        for r, e in zip(rows, ends):
+            self.cache.reserve(r, e)
+        n = len(tokens)
+        single = all(len(t) == 1 for t in tokens) and (want is None or list(want) == list(range(n)))
+        if single and self.use_graphs and self._warm.get(n, 0) >= self.GRAPH_WARMUP and (n in self._graphs or len(self._graphs) < self.MAX_GRAPHS):
+            logits = self._replay([t[0] for t in tokens], start, rows)
+        else:
+            logits = self.model.step(self.cache, StepBatch(self.cache, tokens, start, rows, want, self.cfg.vocab_size))
+            if single:
+                self._warm[n] = self._warm.get(n, 0) + 1
+        self.cache.commit(rows, ends)
+        return logits
+
+    def _replay(self, tokens, start, rows):
+        from .state_cache import StepBatch
+        n = len(tokens)
+        if n not in self._graphs:
+            batch = StepBatch(self.cache, [[t] for t in tokens], start, rows, None, self.cfg.vocab_size)
+            graph = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(graph):
+                logits = self.model.step(self.cache, batch)
+            self._graphs[n] = (graph, batch, logits)
+        graph, batch, logits = self._graphs[n]
+        if min(tokens) < 0 or max(tokens) >= self.cfg.vocab_size:
+            raise ValueError("token id outside the vocabulary")
+        batch.refill(self.cache, tokens, start, rows)
+        graph.replay()
+        return logits
+
     @torch.no_grad()
     def _forward_tree(self, tokens: List[int], parents: List[int], start: int, row: int = 0) -> torch.Tensor:
         """One forward over a TREE of new tokens of cache row ``row``, which holds ``start`` committed tokens.
@@ -117,6 +169,8 @@ class Generator:
         prefix plus its ancestors and itself: one masked attention launch per layer for the whole tree
         (include/oil/inference_opt.h:262-298). Returns logits [len(tokens), vocab]. The caller truncates the row to the
         part it keeps."""
+        if self.stepped:
+            raise NotImplementedError("tree decoding needs a cache that can be rewound; this model keeps recurrent states")
         m, cfg, cache = self.model, self.cfg, self.cache
         T = len(tokens)
         assert 1 <= T <= 64 and all(-1 <= p < i for i, p in enumerate(parents))
@@ -167,8 +221,11 @@ class Generator:
     @torch.no_grad()
     def generate_tokens(self, prompts, max_new_tokens: int = 64, sampling: Optional[SamplingParams] = None, eos_id: Optional[int] = None,
                         on_token: Optional[Callable[[int, List[int]], bool]] = None, stop_tokens: Sequence[int] = ()) -> List[List[int]]:
-        """prompts: [B, S] tensor or list of equal-length id lists. Returns the new tokens per sequence.
-        ``on_token(step, tokens)`` may return False to stop (cooperative stop)."""
+        """prompts: [B, S] tensor or list of equal-length id lists (any lengths for models with a packed step). Returns the new
+        tokens per sequence. ``on_token(step, tokens)`` may return False to stop (cooperative stop)."""
+        lens = [len(p) for p in prompts] if self.stepped and not isinstance(prompts, torch.Tensor) and isinstance(prompts[0], (list, tuple)) else []
+        if len(set(lens)) > 1:
+            return self._generate_unequal(prompts, lens, max_new_tokens, sampling, eos_id, on_token, stop_tokens)
         ids = torch.as_tensor(prompts, dtype=torch.long, device=self.device)
         if ids.dim() == 1:
             ids = ids.unsqueeze(0)
@@ -201,6 +258,33 @@ class Generator:
         sync()
         t2 = time.time()
         self.stats = GenerationStats(prompt_tokens=B * S, new_tokens=sum(len(o) for o in out), prefill_s=t1 - t0, decode_s=t2 - t1)
+        return out
+
+    def _generate_unequal(self, prompts, lens, max_new_tokens, sampling, eos_id, on_token, stop_tokens):
+        """Prompts of different lengths: one packed prefill, then joint decode steps."""
+        B, sampler = len(prompts), Sampler(sampling)
+        for b in range(self.cache.max_batch):
+            self.cache.free(b)
+        rows, out, done = list(range(B)), [[] for _ in range(B)], [False] * B
+        t0 = t1 = time.time()
+        logits = self.step(prompts, [0] * B, rows)
+        for steps in range(1, max_new_tokens + 1):
+            history = None
+            if sampler.p.repetition_penalty != 1.0:
+                seen = [list(p) + o for p, o in zip(prompts, out)]
+                wide = max(len(s) for s in seen)
+                history = torch.tensor([s + [-1] * (wide - len(s)) for s in seen], device=self.device)
+            nxt = sampler.sample(logits, history).tolist()
+            if steps == 1:
+                t1 = time.time()
+            for b, t in enumerate(nxt):
+                if not done[b]:
+                    out[b].append(int(t))
+                    done[b] = (eos_id is not None and t == eos_id) or t in stop_tokens
+            if steps == max_new_tokens or all(done) or (on_token is not None and on_token(steps, [o[-1] for o in out]) is False):
+                break
+            logits = self.step([[t] for t in nxt], [n + steps - 1 for n in lens], rows)
+        self.stats = GenerationStats(prompt_tokens=sum(lens), new_tokens=sum(len(o) for o in out), prefill_s=t1 - t0, decode_s=time.time() - t1)
         return out
 
     def generate(self, prompt: str, max_new_tokens: int = 64, sampling: Optional[SamplingParams] = None) -> str:

@@ -6,6 +6,7 @@ the OIL4 KV format (4-bit indices + fp16 scale per 32 values), appended and read
 KVCache (src/kv_cache.cpp:85-280), PagedKVCacheBase / block tables with a physical-memory cap and
 LRU page eviction (include/oil/kv_cache.h:73-238, src/kv_cache.cpp:286-569), OIL4KVCache
 (src/kv_cache_oil4.cpp:207-362) and the checkpoint / rewind used by speculative decoding.
+``PagedRows`` is the page bookkeeping; the cache of latents and recurrent states (``state_cache.py``) shares it.
 """
 from __future__ import annotations
 
@@ -34,53 +35,48 @@ KV_LEVELS = torch.tensor([-2.7178, -2.0522, -1.5995, -1.2392, -0.9275, -0.6508, 
                           1.5995, 2.0522, 2.7178]) / 2.7178
 
 
-class PagedKVCache:
-    def __init__(self, num_layers: int, num_kv_heads: int, head_dim: int, max_batch: int, max_seq: int, device, fmt: str = "oil4",
-                 num_pages: Optional[int] = None):
-        assert fmt in ("oil4", "bf16") and (fmt == "bf16" or head_dim % 32 == 0)
-        self.L, self.Hkv, self.D, self.fmt = num_layers, num_kv_heads, head_dim, fmt
+class PagedRows:
+    """Host bookkeeping shared by the paged caches: every sequence (cache row) owns 16-token pages of one pool, listed in a
+    page table on the device. A page that a window has left behind can be released early (its entry is then never read)."""
+
+    def __init__(self, max_batch: int, max_seq: int, device, num_pages: Optional[int] = None):
         self.device = torch.device(device)
         self.max_pages = (max_seq + PAGE - 1) // PAGE
         self.num_pages = num_pages or max_batch * self.max_pages
         self.max_batch = max_batch
-        row = head_dim // 2 if fmt == "oil4" else head_dim * 2  # bytes per token per head
-        self.k_pool = [torch.zeros(self.num_pages, num_kv_heads, PAGE, row, dtype=torch.uint8, device=self.device) for _ in range(num_layers)]
-        self.v_pool = [torch.zeros_like(self.k_pool[0]) for _ in range(num_layers)]
-        if fmt == "oil4":
-            self.k_scale = [torch.zeros(self.num_pages, num_kv_heads, PAGE, head_dim // 32, dtype=torch.float16, device=self.device)
-                            for _ in range(num_layers)]
-            self.v_scale = [torch.zeros_like(self.k_scale[0]) for _ in range(num_layers)]
-        else:
-            self.k_scale = self.v_scale = [None] * num_layers
         self.page_table = torch.zeros(max_batch, self.max_pages, dtype=torch.int32, device=self.device)
         self.seq_lens = torch.zeros(max_batch, dtype=torch.int32, device=self.device)
         self._host_lens = [0] * max_batch
         self._host_pages: List[List[int]] = [[] for _ in range(max_batch)]
+        self._released = [0] * max_batch         # leading pages of a row already given back
         self._free = list(range(self.num_pages - 1, -1, -1))
-
-    # ------------------------------------------------------------------ page management (host)
-    def bytes_per_token(self) -> int:
-        per = self.D // 2 + (self.D // 32) * 2 if self.fmt == "oil4" else self.D * 2
-        return 2 * self.L * self.Hkv * per
 
     def reserve(self, b: int, new_len: int):
         """Make sure sequence ``b`` owns pages for ``new_len`` tokens."""
         need = (new_len + PAGE - 1) // PAGE
+        if need > self.max_pages:
+            raise MemoryError(f"sequence of {new_len} tokens is longer than the cache's {self.max_pages * PAGE}")
         pages = self._host_pages[b]
-        added = False
-        while len(pages) < need:
-            if not self._free:
-                raise MemoryError("paged KV cache is out of pages")
-            pages.append(self._free.pop())
-            added = True
-        if added:
+        if need - len(pages) > len(self._free):
+            raise MemoryError("paged KV cache is out of pages")
+        if len(pages) < need:
+            while len(pages) < need:
+                pages.append(self._free.pop())
             self.page_table[b, : len(pages)] = torch.tensor(pages, dtype=torch.int32, device=self.device)
 
     def free(self, b: int):
-        self._free.extend(reversed(self._host_pages[b]))
+        self._free.extend(reversed(self._host_pages[b][self._released[b]:]))
         self._host_pages[b] = []
+        self._released[b] = 0
         self._host_lens[b] = 0
         self.seq_lens[b] = 0
+
+    def release_before(self, b: int, position: int):
+        """Give back the pages of sequence ``b`` that hold only tokens before ``position``."""
+        done = min(position // PAGE, len(self._host_pages[b]))
+        if done > self._released[b]:
+            self._free.extend(self._host_pages[b][self._released[b]:done])
+            self._released[b] = done
 
     def truncate(self, b: int, new_len: int):
         """Rewind a sequence (speculative decoding rolls back rejected drafts)."""
@@ -95,14 +91,40 @@ class PagedKVCache:
         """Exchange two sequences' rows (keeps the active sequences of a continuous batch in rows 0..n-1)."""
         if a == b:
             return
-        self._host_pages[a], self._host_pages[b] = self._host_pages[b], self._host_pages[a]
-        self._host_lens[a], self._host_lens[b] = self._host_lens[b], self._host_lens[a]
+        for x in (self._host_pages, self._host_lens, self._released):
+            x[a], x[b] = x[b], x[a]
         rows = self.page_table[[b, a]].clone()
         self.page_table[[a, b]] = rows
         self.seq_lens[: len(self._host_lens)] = torch.tensor(self._host_lens, dtype=torch.int32, device=self.device)
 
     def lengths(self) -> List[int]:
         return list(self._host_lens)
+
+    def commit(self, batch_ids: List[int], new_lens: List[int]):
+        for b, n in zip(batch_ids, new_lens):
+            self._host_lens[b] = n
+        self.seq_lens[: len(self._host_lens)] = torch.tensor(self._host_lens, dtype=torch.int32, device=self.device)
+
+
+class PagedKVCache(PagedRows):
+    def __init__(self, num_layers: int, num_kv_heads: int, head_dim: int, max_batch: int, max_seq: int, device, fmt: str = "oil4",
+                 num_pages: Optional[int] = None):
+        assert fmt in ("oil4", "bf16") and (fmt == "bf16" or head_dim % 32 == 0)
+        super().__init__(max_batch, max_seq, device, num_pages)
+        self.L, self.Hkv, self.D, self.fmt = num_layers, num_kv_heads, head_dim, fmt
+        row = head_dim // 2 if fmt == "oil4" else head_dim * 2  # bytes per token per head
+        self.k_pool = [torch.zeros(self.num_pages, num_kv_heads, PAGE, row, dtype=torch.uint8, device=self.device) for _ in range(num_layers)]
+        self.v_pool = [torch.zeros_like(self.k_pool[0]) for _ in range(num_layers)]
+        if fmt == "oil4":
+            self.k_scale = [torch.zeros(self.num_pages, num_kv_heads, PAGE, head_dim // 32, dtype=torch.float16, device=self.device)
+                            for _ in range(num_layers)]
+            self.v_scale = [torch.zeros_like(self.k_scale[0]) for _ in range(num_layers)]
+        else:
+            self.k_scale = self.v_scale = [None] * num_layers
+
+    def bytes_per_token(self) -> int:
+        per = self.D // 2 + (self.D // 32) * 2 if self.fmt == "oil4" else self.D * 2
+        return 2 * self.L * self.Hkv * per
 
     # ------------------------------------------------------------------ append / attend
     def append(self, layer: int, k: torch.Tensor, v: torch.Tensor, batch_ids: List[int], start: List[int]):
@@ -159,11 +181,6 @@ class PagedKVCache:
                 x = lv * scale[pages].float().repeat_interleave(32, dim=-1)
             out.append(x.permute(0, 2, 1, 3).reshape(-1, self.Hkv, self.D)[:n])
         return out[0], out[1]
-
-    def commit(self, batch_ids: List[int], new_lens: List[int]):
-        for b, n in zip(batch_ids, new_lens):
-            self._host_lens[b] = n
-        self.seq_lens[: len(self._host_lens)] = torch.tensor(self._host_lens, dtype=torch.int32, device=self.device)
 
     def decode_attention(self, layer: int, q: torch.Tensor, num_heads: int, scale: float, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         """q: [B, >= H*D] token-major rows (one new token per sequence, already appended) -> [B, H*D]."""

@@ -137,7 +137,23 @@ class ContinuousBatching:
     def add_request(self, req: Request):
         self.sched.add(req)
 
+    MAX_PREFILL_TOKENS = 16384      # prompt tokens admitted in one packed step
+
+    def _admit_packed(self):
+        """Models with a packed step: all requests that find a free row are prefilled as one batch of unequal prompts."""
+        while len(self.active) < self.max_batch and self.sched.pending_count():
+            reqs, total = [], 0
+            while len(self.active) + len(reqs) < self.max_batch and self.sched.pending_count() and total < self.MAX_PREFILL_TOKENS:
+                reqs.append(self.sched.next())
+                total += len(reqs[-1].tokens)
+            rows = list(range(len(self.active), len(self.active) + len(reqs)))
+            logits = self.gen.step([r.tokens for r in reqs], [0] * len(reqs), rows)
+            for req, tok in zip(reqs, self.sampler.sample(logits).tolist()):
+                self.active.append(_Active(req, [int(tok)], len(req.tokens), int(tok)))
+
     def _admit(self):
+        if self.gen.stepped:
+            return self._admit_packed()
         while len(self.active) < self.max_batch and self.sched.pending_count():
             req = self.sched.next()
             row = len(self.active)

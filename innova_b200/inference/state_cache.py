@@ -1,0 +1,110 @@
+"""Cache of decoders that mix attention over latents with recurrent layers, and the description of one batch of a step.
+
+``LatentStateCache`` gives every attention run paged latents (16-token pages, one page table for all runs) and every recurrent
+run a slot per sequence: the delta-rule state in fp32 and the ring of the short convolutions' last inputs. A layer that is
+run several times has one pool or one state per run. Slots follow their sequence when rows are swapped, and need no clearing:
+a sequence that starts at position 0 reads neither. When every attention run has a window, the pages that no window can
+reach any more go back to the pool as the sequence grows.
+
+``StepBatch`` packs the new tokens of several sequences (any number each) into one row of tokens and puts everything the
+kernels need to know about them on the device in one copy."""
+from __future__ import annotations
+
+from typing import List, Optional, Sequence
+
+import torch
+
+from .kv_cache import PAGE, PagedRows
+
+
+class StepBatch:
+    """``tokens[i]`` are the next tokens of cache row ``rows[i]``, which holds ``start[i]`` already. ``want``: packed indices
+    whose logits are asked for (None: the last token of every sequence)."""
+
+    def __init__(self, cache: "LatentStateCache", tokens: Sequence[Sequence[int]], start: Sequence[int], rows: Sequence[int],
+                 want: Optional[Sequence[int]] = None, vocab: Optional[int] = None):
+        lens = [len(t) for t in tokens]
+        if not lens or min(lens) < 1:
+            raise ValueError("a step needs at least one token per sequence")
+        if len(set(rows)) != len(rows) or min(rows) < 0 or max(rows) >= cache.max_batch:
+            raise ValueError(f"bad cache rows {list(rows)}")
+        flat = [int(t) for ts in tokens for t in ts]
+        if vocab is not None and not (0 <= min(flat) and max(flat) < vocab):
+            raise ValueError(f"token id outside the vocabulary of {vocab}")
+        self.n, self.T, self.max_len = len(lens), len(flat), max(lens)
+        self.host_rows, self.host_start, self.lens = list(rows), [int(s) for s in start], lens
+        self.max_pos = max(s + n for s, n in zip(self.host_start, lens))
+        self.single = self.max_len == 1              # one token per sequence: the decode kernels
+        self.fresh = not any(self.host_start)        # whole prompts: nothing is read from the cache
+        self.device = cache.device
+        cu = [0]
+        for n in lens:
+            cu.append(cu[-1] + n)
+        if want is None:
+            want = [c - 1 for c in cu[1:]]
+        self.n_want = len(want)
+        self.want_all = list(want) == list(range(self.T))
+        self._buf = torch.empty(4 * self.n + 1 + 3 * self.T + self.n_want, dtype=torch.int32, device=self.device)
+        self._views()
+        self._fill(cache, flat, cu, want)
+
+    def _views(self):
+        sizes = [self.n, self.n, self.n, self.n + 1, self.T, self.T, self.T, self.n_want]
+        self.start, self.rows, self.slots, self.cu, self.ids, self.tok_seq, self.tok_pos, self.want = torch.split(self._buf[:sum(sizes)], sizes)
+
+    def _fill(self, cache, flat, cu, want):
+        seq = [i for i, n in enumerate(self.lens) for _ in range(n)]
+        pos = [s + k for s, n in zip(self.host_start, self.lens) for k in range(n)]
+        slots = [cache.slot_of(r) for r in self.host_rows]
+        host = torch.tensor(self.host_start + self.host_rows + slots + cu + flat + seq + pos + list(want), dtype=torch.int32)
+        self._buf[: host.numel()].copy_(host)
+
+    def refill(self, cache, tokens: Sequence[int], start: Sequence[int], rows: Sequence[int]):
+        """Same shape, next step (one token per sequence): new values in the same device memory (a captured graph reads it)."""
+        self.host_rows, self.host_start = list(rows), [int(s) for s in start]
+        self.max_pos = max(self.host_start) + 1
+        self._fill(cache, [int(t) for t in tokens], list(range(self.n + 1)), range(self.n))
+
+
+class LatentStateCache(PagedRows):
+    """``latents``: (padded rank, window or None) per attention run; ``states``: ``DeltaShape`` per recurrent run."""
+
+    def __init__(self, latents, states, max_batch: int, max_seq: int, device, dtype=torch.bfloat16, num_pages: Optional[int] = None):
+        super().__init__(max_batch, max_seq, device, num_pages)
+        self.windows = [w for _, w in latents]
+        self.dtype = dtype
+        self.latent = [torch.zeros(self.num_pages, PAGE, r, dtype=dtype, device=self.device) for r, _ in latents]
+        self.state = [torch.zeros(max_batch, s.H, s.D, s.Dv, dtype=torch.float32, device=self.device) for s in states]
+        self.ring = [torch.zeros(max_batch, s.taps, s.channels, dtype=torch.float32, device=self.device) for s in states]
+        self._slot = list(range(max_batch))
+        self.reach = None if (not latents or any(not w for w in self.windows)) else max(self.windows)
+
+    def slot_of(self, row: int) -> int:
+        return self._slot[row]
+
+    def bytes_per_token(self) -> int:
+        return sum(p.shape[2] * p.element_size() for p in self.latent)
+
+    def state_bytes(self) -> int:
+        """Bytes of one sequence's recurrent states and convolution inputs."""
+        return sum(t[0].numel() * 4 for t in self.state + self.ring)
+
+    def swap(self, a: int, b: int):
+        super().swap(a, b)
+        self._slot[a], self._slot[b] = self._slot[b], self._slot[a]
+
+    def truncate(self, b: int, new_len: int):
+        if new_len == 0:
+            self.free(b)
+        elif new_len != self._host_lens[b]:
+            raise RuntimeError("a recurrent state cannot be rewound")
+
+    def commit(self, batch_ids: List[int], new_lens: List[int]):
+        for b, n in zip(batch_ids, new_lens):
+            self._host_lens[b] = n
+            if self.reach is not None:      # the next token sees positions > n - reach
+                self.release_before(b, n - self.reach + 1)
+
+    def free(self, b: int):
+        self._free.extend(reversed(self._host_pages[b][self._released[b]:]))
+        self._host_pages[b], self._released[b], self._host_lens[b] = [], 0, 0

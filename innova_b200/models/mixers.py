@@ -1,0 +1,254 @@
+"""Sequence mixers and feed-forward of the layer-list decoders, as modules with fused, padded weights.
+
+A module is built for one set of sizes, loads its tensors by name (``load``), gives them back under the same names
+(``export``), and runs on packed tokens (``run(ctx, h, cache_index)``). ``ctx`` is the step (``StepContext``): it owns the
+projections' precision and the split-K accumulators of decode steps.
+
+Weights of the projections are kept in the model's type with rows padded to 16 bytes; everything that enters a norm, a
+convolution, a decay or a residual is fp32."""
+from __future__ import annotations
+
+from typing import Dict, Optional
+
+import torch
+import torch.nn as nn
+import torch.nn.functional as F
+
+from .. import ops
+from ..ops import delta_rule as dr
+from ..ops import latent_attention as la
+from ..ops.gemm import EPI_ATOMIC, gemm
+from ..ops.hyper import gated_silu, row_buffer
+
+
+def pad_to(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+def frozen(*shape, dtype) -> nn.Parameter:
+    return nn.Parameter(torch.zeros(*shape, dtype=dtype), requires_grad=False)
+
+
+class Proj(nn.Module):
+    """A projection [n, k]; stored [n padded to 8, k padded to 8] so that rows start on 16-byte boundaries."""
+
+    def __init__(self, n: int, k: int, dtype):
+        super().__init__()
+        self.n, self.k = n, k
+        self.weight = frozen(pad_to(n, 8), pad_to(k, 8), dtype=dtype)
+
+
+def put(p: Proj, w: torch.Tensor, row: int = 0):
+    p.weight[row:row + w.shape[0], : w.shape[1]].copy_(w)
+
+
+class StepContext:
+    """Precision and scratch of one forward step. In bf16 decode steps the projections are split over K into fp32
+    accumulators that the consuming kernels leave zeroed (``acc``); otherwise they write tensors of their own."""
+
+    ACC_ROWS = 64
+
+    def __init__(self, model, cache, batch):
+        self.batch, self.cache = batch, cache
+        self.dtype = model.dtype
+        self.acc = model.accumulators(cache.device) if (batch.single and batch.T <= self.ACC_ROWS and model.can_accumulate) else None
+        self.cuda = cache.device.type == "cuda"
+        self.clear: Optional[torch.Tensor] = None      # accumulator columns the running sublayer has to leave zeroed
+
+    def project(self, x: torch.Tensor, p: Proj, out_dtype=None) -> torch.Tensor:
+        """[T, k] -> [T, padded n] (views of the whole padded rows)."""
+        w = p.weight[:, : p.k]
+        if self.cuda and self.dtype == torch.bfloat16:
+            return gemm(x[:, : p.k], w, out_dtype=out_dtype or torch.bfloat16)
+        return F.linear(x[:, : p.k], w).to(out_dtype or self.dtype)
+
+    def project_in(self, x: torch.Tensor, p: Proj) -> torch.Tensor:
+        """First projection of a sublayer."""
+        if self.acc is None:
+            return self.project(x, p)
+        out = self.acc[0][: x.shape[0], : p.weight.shape[0]]
+        gemm(x[:, : p.k], p.weight[:, : p.k], out=out, epilogue=EPI_ATOMIC)
+        self.clear = out
+        return out
+
+    def project_out(self, x: torch.Tensor, p: Proj) -> torch.Tensor:
+        """Last projection of a sublayer: its result goes into the residual."""
+        if self.acc is None:
+            return self.project(x, p)
+        out = self.acc[1][: x.shape[0], : p.weight.shape[0]]
+        gemm(x[:, : p.k], p.weight[:, : p.k], out=out, epilogue=EPI_ATOMIC)
+        return out
+
+
+class LatentAttention(nn.Module):
+    """Attention whose keys and values are linear images of one cached latent per token, optionally windowed.
+
+    Query / value heads are padded to ``Dp`` (64 or 128 where they fit, for the tcgen05 flash kernel) and the latent to ``Rp``
+    with zero weights. Whole bf16 prompts expand keys and values and run flash attention; decode steps, later portions of a
+    prompt and 32-bit models attend in the latent space."""
+
+    kind = "latent_attention"
+
+    def __init__(self, width: int, m: dict, eps: float, dtype, shapes=None):
+        super().__init__()
+        self.H, self.D, self.Dv, self.R = m["heads"], m["dim"], m["vdim"], m["kv_rank"]
+        self.scale, self.eps, self.width = float(m["scale"]), eps, width
+        self.window = (m.get("mask") or {}).get("size")
+        big = max(self.D, self.Dv)
+        self.Dp = 64 if big <= 64 else 128 if big <= 128 else pad_to(big, 16)
+        self.Rp = pad_to(self.R, 16)
+        self.off_c = self.H * self.Dp
+        self.inp = Proj(self.off_c + self.Rp, width, dtype)
+        self.norm = frozen(self.R, dtype=torch.float32)
+        self.uk = frozen(self.H, self.Rp, self.Dp, dtype=dtype)       # per head, latent rows: q' = uk q
+        self.kv = Proj(2 * self.off_c, self.Rp, dtype)                # keys of all heads, then values: expansion of prompts
+        self.out = Proj(width, self.off_c, dtype)
+
+    @property
+    def latent(self):
+        return self.Rp, self.window
+
+    def in_width(self) -> int:
+        return self.inp.weight.shape[0]
+
+    @torch.no_grad()
+    def load(self, t: Dict[str, torch.Tensor], p: str):
+        H, D, Dv, Dp, R = self.H, self.D, self.Dv, self.Dp, self.R
+        self.inp.weight.data[: H * Dp].view(H, Dp, -1)[:, :D, : self.width].copy_(t[p + "q"].view(H, D, self.width))
+        put(self.inp, t[p + "dkv"], self.off_c)
+        self.norm.copy_(t[p + "dkv.norm"])
+        kv = self.kv.weight.data.view(2, H, Dp, -1)
+        kv[0, :, :D, :R].copy_(t[p + "uk"].view(H, D, R))
+        kv[1, :, :Dv, :R].copy_(t[p + "uv"].view(H, Dv, R))
+        self.uk.copy_(kv[0].transpose(1, 2))
+        self.out.weight.data[: self.width].view(self.width, H, Dp)[:, :, :Dv].copy_(t[p + "o"].view(self.width, H, Dv))
+
+    def export(self, p: str) -> Dict[str, torch.Tensor]:
+        H, D, Dv, Dp, R, E = self.H, self.D, self.Dv, self.Dp, self.R, self.width
+        kv = self.kv.weight.view(2, H, Dp, -1)
+        return {p + "q": self.inp.weight[: H * Dp].view(H, Dp, -1)[:, :D, :E].reshape(H * D, E),
+                p + "dkv": self.inp.weight[self.off_c:self.off_c + R, :E], p + "dkv.norm": self.norm,
+                p + "uk": kv[0, :, :D, :R].reshape(H * D, R), p + "uv": kv[1, :, :Dv, :R].reshape(H * Dv, R),
+                p + "o": self.out.weight[:E].view(E, H, Dp)[:, :, :Dv].reshape(E, H * Dv)}
+
+    @staticmethod
+    def shapes(width: int, m: dict, p: str, ranks) -> Dict[str, tuple]:
+        H, D, Dv, R = m["heads"], m["dim"], m["vdim"], m["kv_rank"]
+        return {p + "q": (H * D, width), p + "dkv": (R, width), p + "dkv.norm": (R,), p + "uk": (H * D, R), p + "uv": (H * Dv, R),
+                p + "o": (width, H * Dv)}
+
+    def run(self, ctx: StepContext, h: torch.Tensor, index: int) -> torch.Tensor:
+        b, cache = ctx.batch, ctx.cache
+        pool, T, nq = cache.latent[index], h.shape[0], self.off_c
+        qc = ctx.project_in(h, self.inp)
+        flash = ctx.cuda and ctx.dtype == torch.bfloat16 and b.fresh and not b.single and self.Dp <= 128
+        c, q = la.latent_append(qc, nq, self.R, self.norm, self.eps, pool, cache.page_table, b, want_c=flash,
+                                nq=nq if qc.dtype != pool.dtype else 0)
+        q = qc[:, :nq] if q is None else q
+        if flash:
+            kv = ctx.project(c, self.kv)
+            o = la.packed_flash(q, kv[:, :nq], kv[:, nq:], self.H, self.Dp, self.scale, self.window, b)
+        else:
+            span = min(self.window or cache.max_pages * la.PAGE, cache.max_pages * la.PAGE)
+            lat = la.latent_attend(la.head_proj(q, self.uk), pool, cache.page_table, self.H, self.scale, self.window, b, span)
+            o = la.head_proj(lat, self.kv.weight[nq:2 * nq].view(self.H, self.Dp, self.Rp))
+        return ctx.project_out(o, self.out)
+
+
+class ChannelDelta(nn.Module):
+    """Gated delta rule with short convolutions, a low-rank decay per key channel and a low-rank output gate."""
+
+    kind = "channel_delta"
+
+    def __init__(self, width: int, m: dict, eps: float, dtype, shapes=None):
+        super().__init__()
+        a_rank, g_rank = shapes["a1"][0], shapes["g1"][0]
+        s = self.shape = dr.DeltaShape(m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"], a_rank, g_rank)
+        self.width, self.eps = width, eps
+        self.inp = Proj(s.offsets[6], width, dtype)
+        self.taps = frozen(s.taps, s.channels, dtype=torch.float32)
+        self.a2, self.g2 = Proj(s.H * s.D, a_rank, dtype), Proj(s.H * s.Dv, g_rank, dtype)
+        self.a2t, self.g2t = frozen(a_rank, pad_to(s.H * s.D, 8), dtype=dtype), frozen(g_rank, pad_to(s.H * s.Dv, 8), dtype=dtype)
+        self.A_log, self.dt_bias = frozen(s.H, dtype=torch.float32), frozen(s.H * s.D, dtype=torch.float32)
+        self.norm = frozen(s.Dv, dtype=torch.float32)
+        self.out = Proj(width, s.H * s.Dv, dtype)
+
+    def in_width(self) -> int:
+        return self.inp.weight.shape[0]
+
+    @torch.no_grad()
+    def load(self, t: Dict[str, torch.Tensor], p: str):
+        s, o = self.shape, self.shape.offsets
+        for name, off in zip(("q", "k", "v", "a1", "g1", "b"), o):
+            put(self.inp, t[p + name], off)
+        for name, off in zip(("q", "k", "v"), o):
+            w = t[f"{p}{name}.conv"]
+            self.taps[:, off:off + w.shape[0]].copy_(w.t())
+        put(self.a2, t[p + "a2"])
+        put(self.g2, t[p + "g2"])
+        self.a2t[:, : s.H * s.D].copy_(t[p + "a2"].t())
+        self.g2t[:, : s.H * s.Dv].copy_(t[p + "g2"].t())
+        self.A_log.copy_(t[p + "A_log"])
+        self.dt_bias.copy_(t[p + "dt_bias"])
+        self.norm.copy_(t[p + "norm"])
+        put(self.out, t[p + "o"])
+
+    def export(self, p: str) -> Dict[str, torch.Tensor]:
+        s, o, E = self.shape, self.shape.offsets, self.width
+        rows = {"q": s.Hk * s.D, "k": s.Hk * s.D, "v": s.H * s.Dv, "a1": s.rank_a, "g1": s.rank_g, "b": s.H}
+        out = {p + n: self.inp.weight[off:off + r, :E] for (n, r), off in zip(rows.items(), o)}
+        for n, off in zip("qkv", o):
+            out[f"{p}{n}.conv"] = self.taps[:, off:off + rows[n]].t()
+        out.update({p + "a2": self.a2.weight[: s.H * s.D, : s.rank_a], p + "g2": self.g2.weight[: s.H * s.Dv, : s.rank_g], p + "A_log": self.A_log,
+                    p + "dt_bias": self.dt_bias, p + "norm": self.norm, p + "o": self.out.weight[:E, : s.H * s.Dv]})
+        return out
+
+    @staticmethod
+    def shapes(width: int, m: dict, p: str, ranks) -> Dict[str, tuple]:
+        H, Hk, D, Dv, K, (ra, rg) = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"], ranks
+        out = {p + "b": (H, width), p + "A_log": (H,), p + "norm": (Dv,), p + "a1": (ra, width), p + "a2": (H * D, ra), p + "dt_bias": (H * D,),
+               p + "g1": (rg, width), p + "g2": (H * Dv, rg), p + "o": (width, H * Dv)}
+        for n, ch in (("q", Hk * D), ("k", Hk * D), ("v", H * Dv)):
+            out[p + n], out[f"{p}{n}.conv"] = (ch, width), (ch, K)
+        return out
+
+    def run(self, ctx: StepContext, h: torch.Tensor, index: int) -> torch.Tensor:
+        s, b, cache = self.shape, ctx.batch, ctx.cache
+        proj = ctx.project_in(h, self.inp)
+        args = (self.taps, self.A_log, self.dt_bias, self.norm, self.eps, cache.ring[index], cache.state[index], b)
+        if b.single and s.tile_bytes <= dr.DECODE_MAX_TILE:
+            o = dr.delta_decode(s, proj, self.a2t, self.g2t, *args)
+        else:
+            z = ctx.project(proj[:, s.offsets[3]:], self.a2, torch.float32)
+            gate = ctx.project(proj[:, s.offsets[4]:], self.g2)
+            o = dr.delta_prompt(s, proj, z, gate, *args)
+        return ctx.project_out(o, self.out)
+
+
+class GatedMLP(nn.Module):
+    """W_down (silu(W_gate h) * (W_up h))."""
+
+    def __init__(self, width: int, ff: int, dtype):
+        super().__init__()
+        self.width, self.ff, self.half = width, ff, pad_to(ff, 8)
+        self.inp = Proj(2 * self.half, width, dtype)
+        self.out = Proj(width, ff, dtype)
+
+    def in_width(self) -> int:
+        return self.inp.weight.shape[0]
+
+    @torch.no_grad()
+    def load(self, t, p):
+        put(self.inp, t[p + "gate"])
+        put(self.inp, t[p + "up"], self.half)
+        put(self.out, t[p + "down"])
+
+    def export(self, p):
+        return {p + "gate": self.inp.weight[: self.ff, : self.width], p + "up": self.inp.weight[self.half:self.half + self.ff, : self.width],
+                p + "down": self.out.weight[: self.width, : self.ff]}
+
+    def run(self, ctx: StepContext, h: torch.Tensor, index: int = 0) -> torch.Tensor:
+        return ctx.project_out(gated_silu(ctx.project_in(h, self.inp), self.ff, ctx.dtype), self.out)
+
+
+MIXERS = {c.kind: c for c in (LatentAttention, ChannelDelta)}

@@ -10,6 +10,8 @@ src/autograd_functions.cpp:226-239), gemm_tiled_bias_act (src/math_avx2_tiled.cp
 """
 from __future__ import annotations
 
+import contextlib
+
 import torch
 import torch.nn.functional as F
 
@@ -176,6 +178,20 @@ class _LinearFn(torch.autograd.Function):
         dw = _accumulate_wgrad(weight, dy2, x2) if ctx.needs_input_grad[1] else None
         db = _accumulate_bgrad(bias, dy2, cs) if (ctx.has_bias and ctx.needs_input_grad[2]) else None
         return dx, dw, db, dres, None
+
+
+@contextlib.contextmanager
+def full_fp32_matmul(dtype=torch.float32):
+    """Library products of a 32-bit model in true fp32: no TF32, whatever the process-wide switch says."""
+    mm = torch.backends.cuda.matmul
+    before = mm.allow_tf32
+    if dtype == torch.float32 and before:
+        mm.allow_tf32 = False
+    try:
+        yield
+    finally:
+        if mm.allow_tf32 != before:
+            mm.allow_tf32 = before
 
 
 def _linear_cpu(x, weight, bias, residual, mode):
