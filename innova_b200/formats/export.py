@@ -98,9 +98,10 @@ def load_model_dir(path: str, dtype=torch.bfloat16, device="cpu"):
     from ..models.registry import model_class
     from .importers import TensorFile
     config = read_config_dir(path)
+    cls = model_class(config)
     with TensorFile(os.path.join(path, "model.safetensors"), "safetensors") as f:
         tensors = dict(f.items())
-    return model_class(config).from_tensors(config, tensors, dtype, device)
+    return cls.from_tensors(config, tensors, dtype, device)
 
 
 def load_model(path: str, dtype=torch.float32, device="cpu", ref_layout: bool = False, config: Optional[TransformerConfig] = None):

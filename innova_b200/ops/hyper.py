@@ -70,13 +70,13 @@ def hyper_step(x: torch.Tensor, dtype, prev: Optional[HyperOut] = None, nxt: Opt
 
 
 def _hyper_step_cpu(x, dtype, prev, nxt, ids, table, scale, rows, keep):
-    cur = x
+    cur, E = x, x.shape[2]
     if ids is not None:
-        cur = (table[ids.long()].float() * scale).unsqueeze(1).expand(x.shape).clone()
+        cur = (table[ids.long(), :E].float() * scale).unsqueeze(1).expand(x.shape).clone()
     if rows is not None:
         cur = cur[rows.long()]
     if prev is not None:
-        y = prev.y.float() if rows is None else prev.y[rows.long()].float()
+        y = prev.y[:, :E].float() if rows is None else prev.y[rows.long(), :E].float()
         cur = torch.einsum("nse,st->nte", cur, prev.mix) + prev.out.view(1, -1, 1) * y.unsqueeze(1)
     if keep:
         x.copy_(cur)

@@ -162,12 +162,12 @@ def random_weights(cfg, seed=0, a_rank=12, g_rank=20, dtype=torch.float32):
         p = l + "mix."
         for q in ((1, 2) if L["mlp"] is not None else (1,)):
             w[f"{l}norm{q}"], w[f"{l}norm{q}.b"] = near(E, 1, 0.1), near(E, 0, 0.1)
-            w[f"{l}hc{q}.in"], w[f"{l}hc{q}.out"] = near(S, 1 / S, 0.3), near(S, 1, 0.3)
+            w[f"{l}hc{q}.in"], w[f"{l}hc{q}.out"] = near(S, 1 / S, 0.2), near(S, 1, 0.3)
             w[f"{l}hc{q}.mix"] = torch.eye(S) + 0.2 * torch.randn(S, S, generator=g)
         if L["type"] == "latent_attention":
             H, D, Dv, R = m["heads"], m["dim"], m["vdim"], m["kv_rank"]
-            w[p + "q"], w[p + "dkv"], w[p + "dkv.norm"] = lin(H * D, E, 2.0), lin(R, E), near(R, 1, 0.1)
-            w[p + "uk"], w[p + "uv"], w[p + "o"] = lin(H * D, R, 1.5), lin(H * Dv, R), lin(E, H * Dv)
+            w[p + "q"], w[p + "dkv"], w[p + "dkv.norm"] = lin(H * D, E, 1.3), lin(R, E), near(R, 1, 0.1)
+            w[p + "uk"], w[p + "uv"], w[p + "o"] = lin(H * D, R, 1.3), lin(H * Dv, R), lin(E, H * Dv)
         else:
             H, Hk, D, Dv, K = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
             for n, ch in (("q", Hk * D), ("k", Hk * D), ("v", H * Dv)):
