@@ -4,6 +4,7 @@ parameters / gradients / optimizer state, 64 x 1024 tokens per GPU per step (512
 
     python bench.py --gpus N --steps K --warmup W            # this framework
     python bench.py --impl reference ...                     # the reference (see below)
+    python bench.py --design vebesun                         # another workload: one model design beside its closest models
 
 One JSON line is printed by rank 0. ``value`` is device-timed tokens/s of the whole job (CUDA events,
 max over ranks); ``e2e`` repeats the measurement through ``Trainer.train_step`` with the host-to-device
@@ -88,6 +89,10 @@ def parse():
     ap.add_argument("--engine", default="fsdp3", choices=["fsdp3", "zero2"], help="data-parallel engine at N > 1")
     ap.add_argument("--decode-new", type=int, default=64, help="generated tokens of the decode section (0: skip it)")
     ap.add_argument("--decode-layers", type=int, default=32, help="for debugging only; the reported decode config is 32")
+    ap.add_argument("--design", default=None, choices=["vebesun"], help="instead of the headline workload: throughput of one model design "
+                    "beside the closest models at equal size (bench_vebesun.py)")
+    ap.add_argument("--section", default="all", choices=["all", "model", "kernels"], help="with --design: what to measure")
+    ap.add_argument("--sizes", default="", help="with --design: sizes to measure, with commas")
     return ap.parse_args()
 
 
@@ -327,6 +332,9 @@ def run_ours(args):
 
 def main():
     args = parse()
+    if args.design == "vebesun":
+        import bench_vebesun
+        return bench_vebesun.main(args.section, args.sizes.split(",") if args.sizes else None)
     if args.impl == "reference":
         return run_reference(args)
     run_ours(args)
