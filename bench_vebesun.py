@@ -63,10 +63,10 @@ def model_section(sizes):
     from innova_b200.inference.generator import Generator
     from innova_b200.inference.hybrid_engine import HybridConfig, HybridEngine
     from innova_b200.models import DenseModel, TransformerConfig
+    from innova_b200.models.vebesun import VebesunModel
     dev = torch.device("cuda")
     for size in sizes:
         E, F, H, R, V = SIZES[size]
-        from innova_b200.models.vebesun import VebesunModel
         clocks = ClockSampler(0)
         clocks.start()
         gen = Generator(VebesunModel(vebesun_config(size), seed=0, device=dev), max_batch=64, max_seq=8192 + 64, num_pages=64 * 160)
@@ -196,28 +196,27 @@ def kernel_section(size="2k"):
             c.reserve(i, n)
         b = StepBatch(c, [[0] * n for n in ls], [0] * len(ls), list(range(len(ls))))
         proj, z, gate = rand(T, s.offsets[6]).to(bf), rand(T, H * 128) - 4, rand(T, H * 128).to(bf)
-        taps, A, dt, nw = rand(4, s.channels), rand(H), rand(H * 128), rand(128)
+        taps, A, dt, nw, o = rand(4, s.channels), rand(H), rand(H * 128), rand(128), rand(T, H * 128)
         lib, st, arr = rt.lib(), rt.stream_ptr(), s.c_array()
-        qn, kn, vv, beta, o = rand(T, H * 128), rand(T, H * 128), rand(T, H * 128), rand(T, H).sigmoid(), rand(T, H * 128)
-        g = torch.rand(T, H * 128, device=dev) * 0.1 + 0.9
-        qn, kn = (torch.nn.functional.normalize(a.view(T, H, 128), dim=-1).reshape(T, -1).contiguous() for a in (qn, kn))
+        blocks, vblocks = torch.empty(b.n_chunks * H * s.block_floats, device=dev), torch.empty(b.n_chunks * H * 8 * 256, device=dev)
 
-        def prep():
-            rt.check(lib.inv_delta_prep(proj.data_ptr(), proj.stride(0), 0, taps.data_ptr(), c.ring[0].data_ptr(), b.tok_seq.data_ptr(),
-                                        b.tok_pos.data_ptr(), b.start.data_ptr(), b.slots.data_ptr(), A.data_ptr(), dt.data_ptr(), qn.data_ptr(),
-                                        kn.data_ptr(), vv.data_ptr(), z.data_ptr(), z.stride(0), beta.data_ptr(), T, arr, st), "prep")
+        def chunk():
+            rt.check(lib.inv_delta_chunk(proj.data_ptr(), proj.stride(0), 0, taps.data_ptr(), c.ring[0].data_ptr(), b.chunk_seq.data_ptr(),
+                                         b.cu_chunk.data_ptr(), b.cu.data_ptr(), b.start.data_ptr(), b.slots.data_ptr(), A.data_ptr(), dt.data_ptr(),
+                                         z.data_ptr(), z.stride(0), blocks.data_ptr(), vblocks.data_ptr(), b.n_chunks, arr, st), "chunk")
 
         def scan():
-            rt.check(lib.inv_delta_scan(qn.data_ptr(), kn.data_ptr(), vv.data_ptr(), g.data_ptr(), g.stride(0), beta.data_ptr(), o.data_ptr(),
-                                        c.state[0].data_ptr(), b.cu.data_ptr(), b.start.data_ptr(), b.slots.data_ptr(), b.n, arr, st), "scan")
-        report("delta_scan", f"{name} H{H} 128x128", cold(scan), 5 * T * H * 128 * 4 / 1e9, fp32=4 * 2 * T * H * 128 * 128 / 1e12)
-        report("delta_prep", f"{name} H{H}", cold(prep), T * H * 128 * (3 * 2 + 3 * 4 + 8) / 1e9)
+            rt.check(lib.inv_delta_scan(blocks.data_ptr(), vblocks.data_ptr(), o.data_ptr(), c.state[0].data_ptr(), b.cu_chunk.data_ptr(),
+                                        b.cu.data_ptr(), b.start.data_ptr(), b.slots.data_ptr(), b.n, rt.status_tensor(dev).data_ptr(), arr, st), "scan")
+        moved = (blocks.numel() + vblocks.numel()) * 4 / 1e9
+        report("delta_chunk", f"{name} H{H}", cold(chunk), moved + T * H * 128 * (3 * 2 + 4) / 1e9, fp32=T * H * 128 * (16 * 3 + 12) * 2 / 1e12)
+        report("delta_scan", f"{name} H{H} 128x128", cold(scan), moved + T * H * 128 * 4 / 1e9, fp32=2 * T * H * (3 * 128 * 128 + 2 * 16 * 128) / 1e12)
 
         def hnorm():
             rt.check(lib.inv_gated_head_norm(o.data_ptr(), nw.data_ptr(), gate.data_ptr(), gate.stride(0), 0, proj.data_ptr(), proj.stride(0), 0, T, H,
                                              128, 1e-5, st), "norm")
         report("gated_head_norm", f"{name} H{H}", cold(hnorm), T * H * 128 * 8 / 1e9)
-        del qn, kn, vv, beta, o, g, proj, z, gate
+        del blocks, vblocks, o, proj, z, gate
     for B in (1, 16, 64):
         c = LatentStateCache([], [s], B, 64, dev)
         for i in range(B):

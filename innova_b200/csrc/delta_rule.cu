@@ -2,13 +2,20 @@
 //   S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q          (S: [D, Dv] per head and sequence)
 // with short causal convolutions in front of q, k, v and a gated per-head RMS norm behind o.
 //
-// Prompt path, over packed tokens of several sequences:
-//   delta_prep        one warp per (token, head part): convolution + SiLU, unit norms, decays exp(-exp(A) softplus(z + dt)), beta
+// Prompt path, over packed tokens of several sequences, in chunks of 16 tokens. Inside a chunk that starts from state S0, with
+// G_t the product of the chunk's decays up to token t,
+//   u_t = beta_t (v_t - S0^T (G_t k_t) - sum_{s<t} kap[t, s] u_s)      kap[t, s] = sum_d k_t k_s G_t / G_s   (s < t)
+//   o_t = S0^T (G_t q_t) + sum_{s<=t} P[t, s] u_s                      P[t, s] the same with q_t
+//   S_16 = G_16 S0 + sum_t (G_16 / G_t) k_t u_t^T
+// so the recurrence advances 16 tokens per step and everything that does not involve S0 is computed for all chunks at once:
+//   delta_chunk       one CTA per (chunk, head): convolutions + SiLU, unit norms, decays exp(-exp(A) softplus(z + dt)), the decayed
+//                     keys and queries, kap and P, and with T = (I + diag(beta) kap)^-1 diag(beta) the 16 x 16 maps T and P T.
+//                     Ratios G_t / G_s are running products of decays (never quotients), so strong decays underflow to zero
+//                     and nothing overflows.
 //   conv_tail         keeps the last taps - 1 projection rows of every sequence (a ring of `taps` rows indexed by position)
-//   delta_scan        the recurrence. The rows of a sequence follow one another, so the work of a step is latency: a CTA owns
-//                     a few value columns of one head, LP lanes share a column and keep their D / LP state entries in
-//                     registers, tokens are staged through shared memory 16 at a time with cp.async (double buffered), and
-//                     the arithmetic uses the packed fp32 pair instructions (two products per issue slot).
+//   delta_scan        the sequential part, fp32 FMAs: a CTA owns 16 value columns of one head with the state in shared memory; a
+//                     chunk is two register-tiled products with S0, the two 16 x 16 maps and the update. Chunk blocks arrive by
+//                     bulk copies, double buffered.
 //   gated_head_norm   o / rms(o) * w * sigmoid(gate), cast to the projections' type
 // Decode path: delta_decode does all of it for one token per sequence in one launch, one CTA per (sequence, head): the state
 // tile is read once into shared memory and written once, which bounds the kernel at 8 D Dv bytes per head.
@@ -16,8 +23,6 @@
 #include "inv_api.h"
 
 namespace inv {
-
-typedef unsigned long long u64;
 
 __device__ __forceinline__ float dr_ld(const float* p) { return *p; }
 __device__ __forceinline__ float dr_ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
@@ -32,32 +37,6 @@ __device__ __forceinline__ float dr_silu(float z) { return z / (1.0f + expf(-z))
 __device__ __forceinline__ float dr_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float dr_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
-__device__ __forceinline__ u64 f2_pack(float lo, float hi) {
-  u64 d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-  return d;
-}
-__device__ __forceinline__ float f2_sum(u64 v) {
-  float lo, hi;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
-  return lo + hi;
-}
-__device__ __forceinline__ u64 f2_mul(u64 a, u64 b) {
-  u64 d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-__device__ __forceinline__ u64 f2_fma(u64 a, u64 b, u64 c) {
-  u64 d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ u64 f2_add(u64 a, u64 b) {
-  u64 d;
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-
 // Shapes and column offsets of one mixer. Projection rows hold [q | k | v | low-rank decay | low-rank gate | beta].
 struct DeltaShape {
   int H, Hk, D, Dv, taps;
@@ -66,64 +45,174 @@ struct DeltaShape {
   int rank_a, rank_g;
 };
 
-// Value of convolved channel c (a column of the projection) at the token with packed row t and absolute position pos.
+constexpr int CH = 16;         // tokens per chunk
+constexpr int CH_TAPS = 8;     // longest convolution kept in registers while a thread walks down a chunk
+
+// One (chunk, head) block of floats: decayed keys and queries [D4][16 k | 16 q], keys for the update [16][D4], the maps
+// [16 s][16 T | 16 PT], the chunk's decay [D4]; D4 = D rounded up to 4.
+__host__ __device__ __forceinline__ int block_floats(int D4) { return 32 * D4 + CH * D4 + CH * 32 + D4; }
+
+// Projection value of channel c at absolute position i (i < 0: before the start).
 template <typename T>
-__device__ __forceinline__ float conv_at(const T* proj, int ld, const float* taps_w, const float* ring, const DeltaShape& s, int t, int pos,
-                                         int start, int c) {
-  float a = 0.f;
-  for (int j = 0; j < s.taps; ++j) {
-    const int i = pos - j;
-    if (i < 0) break;
-    const float x = i >= start ? dr_ld(proj + (size_t)(t - j) * ld + c) : ring[(size_t)(i % s.taps) * s.channels + c];
-    a = fmaf(x, taps_w[(size_t)(s.taps - 1 - j) * s.channels + c], a);
-  }
-  return a;
+__device__ __forceinline__ float conv_in(const T* proj, int ld, const float* ring, const DeltaShape& s, long row0, int start, int i, int c) {
+  if (i < 0) return 0.f;
+  return i >= start ? dr_ld(proj + (row0 + (i - start)) * ld + c) : ring[(size_t)(i % s.taps) * s.channels + c];
 }
 
-// ------------------------------------------------------------------------------------------------ prompt: prep
-// Warp roles per token: [0, Hk) q heads, [Hk, 2 Hk) k heads, then H value heads (which also do the decay and beta of the head).
+// ------------------------------------------------------------------------------------------------ prompt: chunks
 template <typename T>
-__global__ void __launch_bounds__(128) delta_prep_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ taps_w,
-                                                         const float* __restrict__ ring0, const int* __restrict__ tok_seq,
-                                                         const int* __restrict__ tok_pos, const int* __restrict__ start,
-                                                         const int* __restrict__ slots, const float* __restrict__ A_log,
-                                                         const float* __restrict__ dt_bias, float* __restrict__ qn, float* __restrict__ kn,
-                                                         float* __restrict__ vv, float* __restrict__ g, int g_ld, float* __restrict__ beta,
-                                                         const DeltaShape s) {
-  const int lane = threadIdx.x & 31, unit = blockIdx.y * 4 + (threadIdx.x >> 5), t = blockIdx.x;
-  if (unit >= 2 * s.Hk + s.H) return;
-  const int seq = tok_seq[t], pos = tok_pos[t], st = start[seq];
+__global__ void __launch_bounds__(256) delta_chunk_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ taps_w,
+                                                          const float* __restrict__ ring0, const int* __restrict__ chunk_seq,
+                                                          const int* __restrict__ cu_chunk, const int* __restrict__ cu,
+                                                          const int* __restrict__ start_, const int* __restrict__ slots,
+                                                          const float* __restrict__ A_log, const float* __restrict__ dt_bias,
+                                                          const float* __restrict__ z, int z_ld, float* __restrict__ blocks,
+                                                          float* __restrict__ vblocks, const DeltaShape s) {
+  extern __shared__ __align__(16) float csm[];
+  __shared__ float kap[CH][CH + 4], P[CH][CH + 4], Tm[CH][CH + 4], beta[CH];
+  const int D = s.D, Dv = s.Dv, D4 = (D + 3) & ~3, cgs = (Dv + 15) / 16;
+  float* q_s = csm;             // [16][D]
+  float* k_s = q_s + CH * D;    // [16][D]
+  float* g_s = k_s + CH * D;    // [16][D]
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, ch = blockIdx.x, h = blockIdx.y;
+  const int seq = chunk_seq[ch], c0 = (ch - cu_chunk[seq]) * CH, start = start_[seq];
+  const long row0 = cu[seq];                       // packed row of the portion's first token (position `start`)
+  const int n = min(CH, cu[seq + 1] - (int)row0 - c0), pos0 = start + c0, hk = h / (s.H / s.Hk);
   const float* ring = ring0 + (size_t)slots[seq] * s.taps * s.channels;
-  if (unit < 2 * s.Hk) {
-    const bool is_q = unit < s.Hk;
-    const int h = is_q ? unit : unit - s.Hk;
-    const int c0 = (is_q ? s.off_q : s.off_k) + h * s.D;
-    float* dst = (is_q ? qn : kn) + ((size_t)t * s.Hk + h) * s.D;
-    float v[8], ss = 0.f;
-#pragma unroll
-    for (int m = 0; m < 8; ++m) {
-      const int d = lane + m * 32;
-      v[m] = d < s.D ? dr_silu(conv_at(proj, ld, taps_w, ring, s, t, pos, st, c0 + d)) : 0.f;
-      ss = fmaf(v[m], v[m], ss);
+  float* blk = blocks + ((size_t)ch * s.H + h) * block_floats(D4);
+  float* vb = vblocks + ((size_t)ch * s.H + h) * cgs * (CH * 16);
+  for (int i = tid; i < 2 * D + cgs * 16; i += 256) {
+    const int v = i - 2 * D;
+    if (v >= Dv) {                                 // padding columns of the last group
+      for (int t = 0; t < CH; ++t) vb[(size_t)(v >> 4) * (CH * 16) + t * 16 + (v & 15)] = 0.f;
+      continue;
     }
-    float r = 1.0f / sqrtf(dr_warp_sum(ss) + 1e-6f);
-    if (is_q) r *= 1.0f / sqrtf((float)s.D);
+    const int c = i < D ? s.off_q + hk * D + i : i < 2 * D ? s.off_k + hk * D + (i - D) : s.off_v + h * Dv + v;
+    float win[CH_TAPS], w[CH_TAPS];                // win[j]: input j + 1 tokens back
+    const bool slide = s.taps <= CH_TAPS;
 #pragma unroll
-    for (int m = 0; m < 8; ++m) {
-      const int d = lane + m * 32;
-      if (d < s.D) dst[d] = v[m] * r;
+    for (int j = 0; j < CH_TAPS; ++j) {
+      w[j] = j < s.taps ? taps_w[(size_t)(s.taps - 1 - j) * s.channels + c] : 0.f;
+      win[j] = j + 1 < s.taps ? conv_in(proj, ld, ring, s, row0, start, pos0 - 1 - j, c) : 0.f;
     }
-    return;
+#pragma unroll
+    for (int t = 0; t < CH; ++t) {
+      const float x = t < n ? dr_ld(proj + (row0 + c0 + t) * ld + c) : 0.f;
+      float a = x * w[0];
+      if (slide) {
+#pragma unroll
+        for (int j = 1; j < CH_TAPS; ++j) a = fmaf(win[j - 1], w[j], a);
+      } else {
+        for (int j = 1; j < s.taps; ++j)
+          a = fmaf(conv_in(proj, ld, ring, s, row0, start, pos0 + t - j, c), taps_w[(size_t)(s.taps - 1 - j) * s.channels + c], a);
+      }
+#pragma unroll
+      for (int j = CH_TAPS - 1; j > 0; --j) win[j] = win[j - 1];
+      win[0] = x;
+      a = t < n ? dr_silu(a) : 0.f;
+      if (i < D) q_s[t * D + i] = a;
+      else if (i < 2 * D) k_s[t * D + i - D] = a;
+      else vb[(size_t)(v >> 4) * (CH * 16) + t * 16 + (v & 15)] = a;
+    }
   }
-  const int h = unit - 2 * s.Hk;
-  for (int d = lane; d < s.Dv; d += 32)
-    vv[((size_t)t * s.H + h) * s.Dv + d] = dr_silu(conv_at(proj, ld, taps_w, ring, s, t, pos, st, s.off_v + h * s.Dv + d));
   const float ea = expf(A_log[h]);
-  for (int d = lane; d < s.D; d += 32) {
-    const size_t i = (size_t)t * g_ld + h * s.D + d;
-    g[i] = expf(-ea * dr_softplus(g[i] + dt_bias[h * s.D + d]));  // in place: the low-rank projection becomes the decay
+  for (int i = tid; i < CH * D; i += 256) {
+    const int t = i / D, d = i % D;
+    g_s[i] = t < n ? expf(-ea * dr_softplus(z[(row0 + c0 + t) * z_ld + h * D + d] + dt_bias[h * D + d])) : 1.f;
   }
-  if (lane == 0) beta[(size_t)t * s.H + h] = dr_sigmoid(dr_ld(proj + (size_t)t * ld + s.off_b + h));
+  if (tid < CH) beta[tid] = tid < n ? dr_sigmoid(dr_ld(proj + (row0 + c0 + tid) * ld + s.off_b + h)) : 0.f;
+  __syncthreads();
+  for (int t = warp; t < CH; t += 8) {             // unit vectors; the query also carries D^-1/2
+    float sq = 0.f, sk = 0.f;
+    for (int d = lane; d < D; d += 32) {
+      sq = fmaf(q_s[t * D + d], q_s[t * D + d], sq);
+      sk = fmaf(k_s[t * D + d], k_s[t * D + d], sk);
+    }
+    const float rq = 1.0f / sqrtf(dr_warp_sum(sq) + 1e-6f) * (1.0f / sqrtf((float)D)), rk = 1.0f / sqrtf(dr_warp_sum(sk) + 1e-6f);
+    for (int d = lane; d < D; d += 32) {
+      q_s[t * D + d] *= rq;
+      k_s[t * D + d] *= rk;
+    }
+  }
+  __syncthreads();
+  // decayed keys and queries, and the keys of the update: a running product down the chunk and one up
+  for (int d = tid; d < D4; d += 256) {
+    float kq[2][CH], G = 1.f;
+    if (d < D) {
+#pragma unroll
+      for (int t = 0; t < CH; ++t) {
+        G *= g_s[t * D + d];
+        kq[0][t] = k_s[t * D + d] * G;
+        kq[1][t] = q_s[t * D + d] * G;
+      }
+    } else {
+#pragma unroll
+      for (int t = 0; t < CH; ++t) kq[0][t] = kq[1][t] = 0.f;
+    }
+#pragma unroll
+    for (int t = 0; t < 2 * CH; t += 4)
+      *reinterpret_cast<float4*>(blk + (size_t)d * 32 + t) =
+          make_float4(kq[t / CH][t % CH], kq[t / CH][t % CH + 1], kq[t / CH][t % CH + 2], kq[t / CH][t % CH + 3]);
+    blk[32 * D4 + CH * D4 + CH * 32 + d] = G;
+    float R = 1.f;
+#pragma unroll
+    for (int t = CH - 1; t >= 0; --t) {
+      blk[32 * D4 + t * D4 + d] = d < D ? k_s[t * D + d] * R : 0.f;
+      if (d < D) R *= g_s[t * D + d];
+    }
+  }
+  // kap and P: 16 lanes per source token s share the channels and walk t upwards with w = k_s * (decays of s + 1 .. t)
+  {
+    const int src = tid >> 4, l = tid & 15;
+    float ak[CH], ap[CH];
+#pragma unroll
+    for (int t = 0; t < CH; ++t) ak[t] = ap[t] = 0.f;
+    for (int d = l; d < D; d += 16) {
+      float w = k_s[src * D + d];
+#pragma unroll
+      for (int t = 0; t < CH; ++t)
+        if (t >= src) {
+          if (t > src) w *= g_s[t * D + d];
+          ak[t] = fmaf(k_s[t * D + d], w, ak[t]);
+          ap[t] = fmaf(q_s[t * D + d], w, ap[t]);
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < CH; ++t) {
+#pragma unroll
+      for (int o = 8; o > 0; o >>= 1) {
+        ak[t] += __shfl_xor_sync(0xffffffffu, ak[t], o);
+        ap[t] += __shfl_xor_sync(0xffffffffu, ap[t], o);
+      }
+      if (l == 0) {
+        kap[t][src] = t > src ? ak[t] : 0.f;
+        P[t][src] = t >= src ? ap[t] : 0.f;
+      }
+    }
+  }
+  __syncthreads();
+  if (tid < CH) {                                  // column tid of T by forward substitution
+    float x[CH];
+#pragma unroll
+    for (int t = 0; t < CH; ++t) {
+      float a = t == tid ? 1.f : 0.f;
+#pragma unroll
+      for (int r = 0; r < CH; ++r)
+        if (r < t) a = fmaf(-kap[t][r], x[r], a);
+      x[t] = beta[t] * a;
+      Tm[t][tid] = x[t];
+    }
+  }
+  __syncthreads();
+  {
+    const int t = tid & 15, c = tid >> 4;          // entry (t, c) of T and of P T
+    float a = 0.f;
+#pragma unroll
+    for (int r = 0; r < CH; ++r) a = fmaf(P[t][r], Tm[r][c], a);
+    float* tw = blk + 32 * D4 + CH * D4 + c * 32;
+    tw[t] = Tm[t][c];
+    tw[CH + t] = a;
+  }
 }
 
 template <typename T>
@@ -138,163 +227,208 @@ __global__ void __launch_bounds__(256) conv_tail_kernel(const T* __restrict__ pr
 }
 
 // ------------------------------------------------------------------------------------------------ prompt: scan
-constexpr int SCAN_CT = 16;  // tokens per staged chunk
+constexpr int SC_THREADS = 128;
+constexpr int SC_COLS = 16;
 
-template <int DP, int LP, int THREADS>
-struct ScanSmem {
-  static constexpr int COLS = THREADS / LP;
-  static constexpr int ROW = 3 * DP;                                     // q | k | g of one token
-  static constexpr int BUF = SCAN_CT * (ROW + COLS + 4);                 // + values and (padded) beta
-  static constexpr int BYTES = (2 * BUF + SCAN_CT * COLS) * 4;           // two buffers and the outputs of a chunk
-};
-
-// 16-byte (vec) or 4-byte asynchronous copy into shared memory.
-__device__ __forceinline__ void cp16(float* dst, const float* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp4(float* dst, const float* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-
-template <int DP, int LP, int THREADS>
-__global__ void __launch_bounds__(THREADS) delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn,
-                                                             const float* __restrict__ vv, const float* __restrict__ g, int g_ld,
-                                                             const float* __restrict__ beta, float* __restrict__ o, float* __restrict__ state0,
-                                                             const int* __restrict__ cu, const int* __restrict__ start,
-                                                             const int* __restrict__ slots, int H, int Hk, int D, int Dv) {
-  using L = ScanSmem<DP, LP, THREADS>;
-  constexpr int COLS = L::COLS, NP = DP / LP / 2;  // packed pairs of state per lane
+__global__ void __launch_bounds__(SC_THREADS) delta_scan_kernel(const float* __restrict__ blocks, const float* __restrict__ vblocks,
+                                                                float* __restrict__ o, float* __restrict__ state0,
+                                                                const int* __restrict__ cu_chunk, const int* __restrict__ cu,
+                                                                const int* __restrict__ start, const int* __restrict__ slots, int H, int D, int Dv,
+                                                                int* status) {
   extern __shared__ __align__(16) float sm[];
-  float* o_s = sm + 2 * L::BUF;
-  const int tid = threadIdx.x, part = tid % LP, cl = tid / LP;
-  const int h = blockIdx.y, seq = blockIdx.z, hk = h / (H / Hk);
-  const int col0 = blockIdx.x * COLS, col = col0 + cl;
-  const bool live = col < Dv;
-  const int t0 = cu[seq], n = cu[seq + 1] - t0;
+  __shared__ uint64_t full[2];
+  __shared__ int abort_flag;
+  const int D4 = (D + 3) & ~3, bf = block_floats(D4), cgs = gridDim.x;
+  const int stage_floats = bf + CH * SC_COLS;
+  float* S = sm;                              // [D4][16]
+  float* part = S + D4 * SC_COLS;             // [4 warps][32][16]
+  float* R = part + 4 * 32 * SC_COLS;         // [16][16]
+  float* U = R + CH * SC_COLS;                // [16][16]
+  float* buf = U + CH * SC_COLS;              // [2][block | values]
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int cg = blockIdx.x, h = blockIdx.y, seq = blockIdx.z, col0 = cg * SC_COLS;
+  const int ch0 = cu_chunk[seq], nc = cu_chunk[seq + 1] - ch0, row0 = cu[seq], len = cu[seq + 1] - row0;
   float* state = state0 + ((size_t)slots[seq] * H + h) * (size_t)D * Dv;
-  // entry of pair j of this lane: d = 4 (part + LP (j / 2)) + 2 (j % 2) + {0, 1}
-  u64 S[NP];
-#pragma unroll
-  for (int j = 0; j < NP; ++j) {
-    const int d = 4 * (part + LP * (j / 2)) + 2 * (j % 2);
-    float a = 0.f, b = 0.f;
-    if (live && start[seq] > 0) {
-      if (d < D) a = state[(size_t)d * Dv + col];
-      if (d + 1 < D) b = state[(size_t)(d + 1) * Dv + col];
-    }
-    S[j] = f2_pack(a, b);
-  }
-  for (int i = tid; i < 2 * L::BUF; i += THREADS) sm[i] = 0.f;  // channels beyond D and columns beyond Dv stay zero
-  __syncthreads();
-  const bool vec = D % 4 == 0;
-  auto stage = [&](int c, int buf) {
-    float* b = sm + buf * L::BUF;
-    const int m = min(SCAN_CT, n - c * SCAN_CT);
-    const size_t tb = (size_t)t0 + (size_t)c * SCAN_CT;
-    if (vec) {
-      const int per = D / 4, tot = m * per;
-      for (int i = tid; i < tot; i += THREADS) {
-        const int r = i / per, d = (i % per) * 4;
-        const size_t t = tb + r;
-        cp16(b + r * L::ROW + d, qn + (t * Hk + hk) * D + d);
-        cp16(b + r * L::ROW + DP + d, kn + (t * Hk + hk) * D + d);
-        cp16(b + r * L::ROW + 2 * DP + d, g + t * g_ld + (size_t)h * D + d);
-      }
-    } else {
-      for (int i = tid; i < m * D; i += THREADS) {
-        const int r = i / D, d = i % D;
-        const size_t t = tb + r;
-        cp4(b + r * L::ROW + d, qn + (t * Hk + hk) * D + d);
-        cp4(b + r * L::ROW + DP + d, kn + (t * Hk + hk) * D + d);
-        cp4(b + r * L::ROW + 2 * DP + d, g + t * g_ld + (size_t)h * D + d);
-      }
-    }
-    float* vb = b + SCAN_CT * L::ROW;
-    for (int i = tid; i < m * COLS; i += THREADS) {
-      const int r = i / COLS, c2 = i % COLS;
-      if (col0 + c2 < Dv) cp4(vb + r * COLS + c2, vv + ((tb + r) * H + h) * Dv + col0 + c2);
-    }
-    if (tid < m) cp4(vb + SCAN_CT * COLS + tid, beta + (tb + tid) * H + h);
-    asm volatile("cp.async.commit_group;" ::: "memory");
+  auto stage = [&](int c) {                   // thread 0
+    float* b = buf + (c & 1) * stage_floats;
+    const size_t id = (size_t)(ch0 + c) * H + h;
+    mbar_expect_tx(&full[c & 1], (uint32_t)stage_floats * 4u);
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(b)),
+                 "l"(blocks + id * bf), "r"((uint32_t)bf * 4u), "r"(smem_u32(&full[c & 1]))
+                 : "memory");
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(b + bf)),
+                 "l"(vblocks + (id * cgs + cg) * (CH * SC_COLS)), "r"((uint32_t)(CH * SC_COLS) * 4u), "r"(smem_u32(&full[c & 1]))
+                 : "memory");
   };
-  const int nc = (n + SCAN_CT - 1) / SCAN_CT;
-  if (nc > 0) stage(0, 0);
+  if (tid == 0) {
+    abort_flag = 0;
+    mbar_init(&full[0], 1);
+    mbar_init(&full[1], 1);
+    fence_barrier_init();
+    if (nc > 0) stage(0);
+  }
+  for (int i = tid; i < D4 * SC_COLS; i += SC_THREADS) {
+    const int d = i / SC_COLS, c = col0 + i % SC_COLS;
+    S[i] = (start[seq] > 0 && d < D && c < Dv) ? state[(size_t)d * Dv + c] : 0.f;
+  }
+  __syncthreads();
+  const int r = tid >> 2, c4 = (tid & 3) * 4;       // phases 2 and 3: row of [16 T | 16 PT] and four columns
+  const int tg = lane >> 2;                         // phase 1: four of the 32 rows, columns c4
+  bool ok = true;
   for (int c = 0; c < nc; ++c) {
-    if (c + 1 < nc) {
-      stage(c + 1, (c + 1) & 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    if (tid == 0 && c + 1 < nc) stage(c + 1);       // its buffer was last read before the barrier that ended chunk c - 1
+    ok = mbar_wait(&full[c & 1], (c >> 1) & 1, &abort_flag, status, ERR_WAIT_FULL);
+    const float* b = buf + (c & 1) * stage_floats;
+    // 1. [keys; queries] x S0, channels split over the warps
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+#pragma unroll 8
+    for (int d = warp; d < D4; d += 4) {
+      const float4 a = *reinterpret_cast<const float4*>(b + d * 32 + tg * 4);
+      const float4 x = *reinterpret_cast<const float4*>(S + d * SC_COLS + c4);
+      const float av[4] = {a.x, a.y, a.z, a.w}, xv[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], xv[j], acc[i][j]);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      *reinterpret_cast<float4*>(part + (warp * 32 + tg * 4 + i) * SC_COLS + c4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+    if (!__syncthreads_and(ok)) break;
+    // 2. sum over the warps; rows 0..15 become v - S0^T k, rows 16..31 stay here for the outputs
+    float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+      const float4 x = *reinterpret_cast<const float4*>(part + (w * 32 + r) * SC_COLS + c4);
+      y.x += x.x; y.y += x.y; y.z += x.z; y.w += x.w;
+    }
+    if (r < CH) {
+      const float4 v = *reinterpret_cast<const float4*>(b + bf + r * SC_COLS + c4);
+      *reinterpret_cast<float4*>(R + r * SC_COLS + c4) = make_float4(v.x - y.x, v.y - y.y, v.z - y.z, v.w - y.w);
+      y = make_float4(0.f, 0.f, 0.f, 0.f);
     }
     __syncthreads();
-    const float* b = sm + (c & 1) * L::BUF;
-    const float* vb = b + SCAN_CT * L::ROW;
-    const int m = min(SCAN_CT, n - c * SCAN_CT);
-    for (int r = 0; r < m; ++r) {
-      const ulonglong2* q2 = reinterpret_cast<const ulonglong2*>(b + r * L::ROW);
-      const ulonglong2* k2 = reinterpret_cast<const ulonglong2*>(b + r * L::ROW + DP);
-      const ulonglong2* g2 = reinterpret_cast<const ulonglong2*>(b + r * L::ROW + 2 * DP);
-      u64 kk[NP], acc[4] = {0, 0, 0, 0};
+    // 3. U = T R (rows 0..15), O = S0^T q + P T R (rows 16..31)
+    const float* tw = b + 32 * D4 + CH * D4 + r;
 #pragma unroll
-      for (int j = 0; j < NP / 2; ++j) {
-        const ulonglong2 gg = g2[part + LP * j], kv = k2[part + LP * j];
-        kk[2 * j] = kv.x;
-        kk[2 * j + 1] = kv.y;
-        S[2 * j] = f2_mul(S[2 * j], gg.x);
-        S[2 * j + 1] = f2_mul(S[2 * j + 1], gg.y);
-        acc[(2 * j) & 3] = f2_fma(S[2 * j], kv.x, acc[(2 * j) & 3]);
-        acc[(2 * j + 1) & 3] = f2_fma(S[2 * j + 1], kv.y, acc[(2 * j + 1) & 3]);
-      }
-      float rk = f2_sum(f2_add(f2_add(acc[0], acc[1]), f2_add(acc[2], acc[3])));
-#pragma unroll
-      for (int w = 1; w < LP; w <<= 1) rk += __shfl_xor_sync(0xffffffffu, rk, w);
-      const float u = vb[SCAN_CT * COLS + r] * (vb[r * COLS + cl] - rk);
-      const u64 uu = f2_pack(u, u);
-      acc[0] = acc[1] = acc[2] = acc[3] = 0;
-#pragma unroll
-      for (int j = 0; j < NP / 2; ++j) {
-        const ulonglong2 qv = q2[part + LP * j];
-        S[2 * j] = f2_fma(kk[2 * j], uu, S[2 * j]);
-        S[2 * j + 1] = f2_fma(kk[2 * j + 1], uu, S[2 * j + 1]);
-        acc[(2 * j) & 3] = f2_fma(S[2 * j], qv.x, acc[(2 * j) & 3]);
-        acc[(2 * j + 1) & 3] = f2_fma(S[2 * j + 1], qv.y, acc[(2 * j + 1) & 3]);
-      }
-      float ov = f2_sum(f2_add(f2_add(acc[0], acc[1]), f2_add(acc[2], acc[3])));
-#pragma unroll
-      for (int w = 1; w < LP; w <<= 1) ov += __shfl_xor_sync(0xffffffffu, ov, w);
-      if (part == 0) o_s[r * COLS + cl] = ov;
+    for (int k = 0; k < CH; ++k) {
+      const float w = tw[k * 32];
+      const float4 x = *reinterpret_cast<const float4*>(R + k * SC_COLS + c4);
+      y.x = fmaf(w, x.x, y.x); y.y = fmaf(w, x.y, y.y); y.z = fmaf(w, x.z, y.z); y.w = fmaf(w, x.w, y.w);
     }
-    __syncthreads();  // everyone is done with this buffer, and the outputs are complete
-    for (int i = tid; i < m * COLS; i += THREADS) {
-      const int r = i / COLS, c2 = i % COLS;
-      if (col0 + c2 < Dv) o[(((size_t)t0 + (size_t)c * SCAN_CT + r) * H + h) * Dv + col0 + c2] = o_s[i];
+    if (r < CH) {
+      *reinterpret_cast<float4*>(U + r * SC_COLS + c4) = y;
+    } else {
+      const int t = c * CH + r - CH;
+      if (t < len) {
+        float* dst = o + ((size_t)(row0 + t) * H + h) * Dv + col0 + c4;
+        const float yv[4] = {y.x, y.y, y.z, y.w};
+        if (Dv % 4 == 0 && col0 + c4 < Dv) *reinterpret_cast<float4*>(dst) = y;
+        else if (Dv % 4)
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if (col0 + c4 + j < Dv) dst[j] = yv[j];
+      }
     }
+    __syncthreads();
+    // 4. S <- G S + K^T U, four channels by four columns per thread
+    const float* kout = b + 32 * D4;
+    const float* gend = kout + CH * D4 + CH * 32;
+    for (int d = (tid >> 2) * 4; d < D4; d += SC_THREADS) {
+      float a4[4][4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float g = gend[d + i];
+        const float4 x = *reinterpret_cast<const float4*>(S + (d + i) * SC_COLS + c4);
+        a4[i][0] = g * x.x; a4[i][1] = g * x.y; a4[i][2] = g * x.z; a4[i][3] = g * x.w;
+      }
+#pragma unroll
+      for (int t = 0; t < CH; ++t) {
+        const float4 a = *reinterpret_cast<const float4*>(kout + t * D4 + d);
+        const float4 x = *reinterpret_cast<const float4*>(U + t * SC_COLS + c4);
+        const float av[4] = {a.x, a.y, a.z, a.w}, xv[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) a4[i][j] = fmaf(av[i], xv[j], a4[i][j]);
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(S + (d + i) * SC_COLS + c4) = make_float4(a4[i][0], a4[i][1], a4[i][2], a4[i][3]);
+    }
+    __syncthreads();
   }
-  if (live) {
-#pragma unroll
-    for (int j = 0; j < NP; ++j) {
-      const int d = 4 * (part + LP * (j / 2)) + 2 * (j % 2);
-      float a, bb;
-      asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(bb) : "l"(S[j]));
-      if (d < D) state[(size_t)d * Dv + col] = a;
-      if (d + 1 < D) state[(size_t)(d + 1) * Dv + col] = bb;
-    }
+  if (!__syncthreads_and(ok)) {  // a copy never arrived: leave the ones in flight a bounded time before the shared memory goes away
+    const uint64_t t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 2000000ull) __nanosleep(1000);
+    return;
+  }
+  for (int i = tid; i < D4 * SC_COLS; i += SC_THREADS) {
+    const int d = i / SC_COLS, c = col0 + i % SC_COLS;
+    if (d < D && c < Dv) state[(size_t)d * Dv + c] = S[i];
   }
 }
 
 // ------------------------------------------------------------------------------------------------ prompt: output norm
-template <typename TG, typename TO>
-__global__ void __launch_bounds__(128) gated_head_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, const TG* __restrict__ gate,
-                                                              int gate_ld, TO* __restrict__ out, int out_ld, int H, int Dv, float eps) {
-  const int lane = threadIdx.x & 31, h = blockIdx.y * 4 + (threadIdx.x >> 5);
-  const size_t t = blockIdx.x;
-  if (h >= H) return;
-  const float* r = o + (t * H + h) * Dv;
+__device__ __forceinline__ void dr_ld4(const float* p, float* f) {
+  const float4 v = *reinterpret_cast<const float4*>(p);
+  f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+__device__ __forceinline__ void dr_ld4(const __nv_bfloat16* p, float* f) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
+  f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
+}
+__device__ __forceinline__ void dr_st4(float* p, const float* f) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+__device__ __forceinline__ void dr_st4(__nv_bfloat16* p, const float* f) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
+}
+
+// One warp per (token, head). V = 4: the row stays in registers (Dv <= 256, Dv % 4 == 0); V = 1: any Dv.
+template <typename TG, typename TO, int V>
+__global__ void __launch_bounds__(256) gated_head_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, const TG* __restrict__ gate,
+                                                              int gate_ld, TO* __restrict__ out, int out_ld, int H, int Dv, float eps, long n_rows) {
+  const int lane = threadIdx.x & 31;
+  const long i = (long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (i >= n_rows) return;
+  const size_t t = i / H;
+  const int h = (int)(i % H);
+  const float* r = o + (size_t)i * Dv;
+  const TG* gp = gate + t * gate_ld + h * Dv;
+  TO* op = out + t * out_ld + h * Dv;
   float ss = 0.f;
-  for (int d = lane; d < Dv; d += 32) ss = fmaf(r[d], r[d], ss);
-  const float inv = 1.0f / sqrtf(dr_warp_sum(ss) / (float)Dv + eps);
-  for (int d = lane; d < Dv; d += 32)
-    dr_st(out + t * out_ld + h * Dv + d, r[d] * inv * w[d] * dr_sigmoid(dr_ld(gate + t * gate_ld + h * Dv + d)));
+  if (V == 4) {
+    float x[2][4], g[2][4];
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      const int d = (lane + m * 32) * 4;
+      if (d < Dv) {
+        dr_ld4(r + d, x[m]);
+        dr_ld4(gp + d, g[m]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) ss = fmaf(x[m][j], x[m][j], ss);
+      }
+    }
+    const float inv = 1.0f / sqrtf(dr_warp_sum(ss) / (float)Dv + eps);
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      const int d = (lane + m * 32) * 4;
+      if (d < Dv) {
+        float y[4];
+        dr_ld4(w + d, y);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[j] = x[m][j] * inv * y[j] * dr_sigmoid(g[m][j]);
+        dr_st4(op + d, y);
+      }
+    }
+  } else {
+    for (int d = lane; d < Dv; d += 32) ss = fmaf(r[d], r[d], ss);
+    const float inv = 1.0f / sqrtf(dr_warp_sum(ss) / (float)Dv + eps);
+    for (int d = lane; d < Dv; d += 32) dr_st(op + d, r[d] * inv * w[d] * dr_sigmoid(dr_ld(gp + d)));
+  }
 }
 
 // ------------------------------------------------------------------------------------------------ decode, one launch
@@ -302,7 +436,7 @@ __global__ void __launch_bounds__(128) gated_head_norm_kernel(const float* __res
 // memory while the convolutions, norms and low-rank products run, it is updated in place and a bulk copy writes it back.
 // Row groups of threads walk the tile (VEC value columns per thread); three tiles of 128 x 128 share an SM.
 constexpr int DD_THREADS = 256;
-constexpr int DD_MAX_TILE = 200 * 1024;
+constexpr int DD_MAX_TILE = 192 * 1024;
 
 template <typename T, typename TW, typename TO, int VEC>
 __global__ void __launch_bounds__(DD_THREADS) delta_decode_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ taps_w,
@@ -328,6 +462,7 @@ __global__ void __launch_bounds__(DD_THREADS) delta_decode_kernel(const T* __res
   float* lr = gate_s + Dv;               // [rank_a + rank_g]
   float* ws = lr + s.rank_a + s.rank_g;  // [2 * NW]
   float* red = ws + 2 * NW;              // [groups * Dv]
+  float* low = red + groups * Dv;        // [NW][D + Dv]
   const int pos = pos_[b], slot = slots[b], hk = h / (s.H / s.Hk);
   const T* row = proj + (size_t)b * ld;
   float* ring = ring0 + (size_t)slot * s.taps * s.channels;
@@ -373,21 +508,52 @@ __global__ void __launch_bounds__(DD_THREADS) delta_decode_kernel(const T* __res
   float nq2 = 0.f, nk2 = 0.f;
   for (int i = 0; i < NW; ++i) { nq2 += ws[i]; nk2 += ws[NW + i]; }
   const float rq = 1.0f / sqrtf(nq2 + 1e-6f) * (1.0f / sqrtf((float)D)), rk = 1.0f / sqrtf(nk2 + 1e-6f);
-  // low-rank decay and output gate (their second matrices are stored transposed: [rank, heads * channels])
+  // low-rank decay and output gate (their second matrices are stored transposed: [rank, heads * channels]): a thread adds VW
+  // neighbouring channels over every eighth rank row, and the eight partial sums meet in shared memory
   const float ea = expf(A_log[h]);
+  {
+    constexpr int VW = 16 / sizeof(TW);
+    const int dg = (D + VW - 1) / VW, vg = (Dv + VW - 1) / VW;
+    const bool vec = D % VW == 0 && Dv % VW == 0;   // rows are 16-byte multiples, so every piece is aligned
+    for (int p = lane; p < dg + vg; p += 32) {
+      const bool is_a = p < dg;
+      const int c = (is_a ? p : p - dg) * VW, width = is_a ? D : Dv, rank = is_a ? s.rank_a : s.rank_g, ldw = is_a ? a2_ld : g2_ld;
+      const TW* w = (is_a ? a2t + h * D : g2t + h * Dv) + c;
+      const float* f = lr + (is_a ? 0 : s.rank_a);
+      float a[VW];
+#pragma unroll
+      for (int j = 0; j < VW; ++j) a[j] = 0.f;
+      if (vec) {
+#pragma unroll 8
+        for (int r = warp; r < rank; r += NW) {
+          float x[VW];
+#pragma unroll
+          for (int j = 0; j < VW; j += 4) dr_ld4(w + (size_t)r * ldw + j, x + j);
+          const float fr = f[r];
+#pragma unroll
+          for (int j = 0; j < VW; ++j) a[j] = fmaf(x[j], fr, a[j]);
+        }
+      } else {
+        for (int r = warp; r < rank; r += NW)
+#pragma unroll
+          for (int j = 0; j < VW; ++j)
+            if (c + j < width) a[j] = fmaf(dr_ld(w + (size_t)r * ldw + j), f[r], a[j]);
+      }
+#pragma unroll
+      for (int j = 0; j < VW; ++j)
+        if (c + j < width) low[warp * (D + Dv) + (is_a ? 0 : D) + c + j] = a[j];
+    }
+  }
+  __syncthreads();
   for (int d = tid; d < D + Dv; d += DD_THREADS) {
     float a = 0.f;
+#pragma unroll
+    for (int i = 0; i < NW; ++i) a += low[i * (D + Dv) + d];
     if (d < D) {
-      const TW* w = a2t + h * D + d;
-#pragma unroll 8
-      for (int r = 0; r < s.rank_a; ++r) a = fmaf(dr_ld(w + (size_t)r * a2_ld), lr[r], a);
       g_s[d] = expf(-ea * dr_softplus(a + dt_bias[h * D + d]));
       q_s[d] *= rq;
       k_s[d] *= rk;
     } else {
-      const TW* w = g2t + h * Dv + (d - D);
-#pragma unroll 8
-      for (int r = 0; r < s.rank_g; ++r) a = fmaf(dr_ld(w + (size_t)r * g2_ld), lr[s.rank_a + r], a);
       gate_s[d - D] = dr_sigmoid(a);
     }
   }
@@ -483,7 +649,8 @@ static int launch_delta_decode(const void* proj, int ld, const float* taps_w, fl
                                const float* A_log, const float* dt_bias, const void* a2t, int a2_ld, const void* g2t, int g2_ld,
                                const float* norm_w, float eps, void* out, int out_ld, int B, int* status, const DeltaShape& s, cudaStream_t st) {
   const int lanes_per_row = (s.Dv / VEC + 31) & ~31, groups = DD_THREADS / lanes_per_row;
-  const size_t smem = (size_t)(((s.D * s.Dv + 3) & ~3) + 3 * s.D + 2 * s.Dv + s.rank_a + s.rank_g + 2 * (DD_THREADS / 32) + groups * s.Dv) * 4;
+  const size_t smem = (size_t)(((s.D * s.Dv + 3) & ~3) + 3 * s.D + 2 * s.Dv + s.rank_a + s.rank_g + 2 * (DD_THREADS / 32) + groups * s.Dv +
+                                (DD_THREADS / 32) * (s.D + s.Dv)) * 4;
   if (s.D * s.Dv * 4 > DD_MAX_TILE || smem > 226 * 1024) return -ERR_BAD_ARG;
   static bool configured = false;
   if (!configured) {
@@ -498,22 +665,6 @@ static int launch_delta_decode(const void* proj, int ld, const float* taps_w, fl
   return e == cudaSuccess ? 0 : -(int)e;
 }
 
-template <int DP, int LP, int THREADS>
-static int launch_scan(const float* qn, const float* kn, const float* vv, const float* g, int g_ld, const float* beta, float* o, float* state,
-                       const int* cu, const int* start, const int* slots, int n_seq, const DeltaShape& s, cudaStream_t st) {
-  using L = ScanSmem<DP, LP, THREADS>;
-  static bool configured = false;
-  if (!configured) {
-    const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<DP, LP, THREADS>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::BYTES);
-    if (e != cudaSuccess) return -(int)e;
-    configured = true;
-  }
-  const dim3 grid((s.Dv + L::COLS - 1) / L::COLS, s.H, n_seq);
-  delta_scan_kernel<DP, LP, THREADS><<<grid, THREADS, L::BYTES, st>>>(qn, kn, vv, g, g_ld, beta, o, state, cu, start, slots, s.H, s.Hk, s.D, s.Dv);
-  const cudaError_t e = cudaGetLastError();
-  return e == cudaSuccess ? 0 : -(int)e;
-}
-
 static bool delta_shape_ok(const DeltaShape& s) {
   return s.H > 0 && s.Hk > 0 && s.H % s.Hk == 0 && s.D > 0 && s.D <= 256 && s.Dv > 0 && s.Dv <= 256 && s.taps > 0;
 }
@@ -523,20 +674,28 @@ static bool delta_shape_ok(const DeltaShape& s) {
 using namespace inv;
 
 // `shape`: the 14 ints of DeltaShape. proj_f32: projection rows are fp32, else bf16.
-extern "C" int inv_delta_prep(const void* proj, int ld, int proj_f32, const float* taps_w, const float* ring, const int* tok_seq, const int* tok_pos,
-                              const int* start, const int* slots, const float* A_log, const float* dt_bias, float* qn, float* kn, float* vv,
-                              float* g, int g_ld, float* beta, int T, const int* shape, void* stream) {
+extern "C" int inv_delta_chunk(const void* proj, int ld, int proj_f32, const float* taps_w, const float* ring, const int* chunk_seq,
+                               const int* cu_chunk, const int* cu, const int* start, const int* slots, const float* A_log, const float* dt_bias,
+                               const float* z, int z_ld, float* blocks, float* vblocks, int n_chunks, const int* shape, void* stream) {
   const DeltaShape s = *reinterpret_cast<const DeltaShape*>(shape);
   if (!delta_shape_ok(s)) return -ERR_BAD_ARG;
-  if (T <= 0) return 0;
-  const dim3 grid(T, (2 * s.Hk + s.H + 3) / 4);
+  if (n_chunks <= 0) return 0;
+  const dim3 grid(n_chunks, s.H);
+  const int smem = 3 * CH * s.D * 4;   // at most 48 KB
   cudaStream_t st = (cudaStream_t)stream;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(delta_chunk_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 3 * CH * 256 * 4);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_chunk_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 3 * CH * 256 * 4);
+    if (e != cudaSuccess) return -(int)e;
+    configured = true;
+  }
   if (proj_f32)
-    delta_prep_kernel<float><<<grid, 128, 0, st>>>((const float*)proj, ld, taps_w, ring, tok_seq, tok_pos, start, slots, A_log, dt_bias, qn, kn, vv, g,
-                                                   g_ld, beta, s);
+    delta_chunk_kernel<float><<<grid, 256, smem, st>>>((const float*)proj, ld, taps_w, ring, chunk_seq, cu_chunk, cu, start, slots, A_log, dt_bias, z,
+                                                       z_ld, blocks, vblocks, s);
   else
-    delta_prep_kernel<__nv_bfloat16><<<grid, 128, 0, st>>>((const __nv_bfloat16*)proj, ld, taps_w, ring, tok_seq, tok_pos, start, slots, A_log,
-                                                           dt_bias, qn, kn, vv, g, g_ld, beta, s);
+    delta_chunk_kernel<__nv_bfloat16><<<grid, 256, smem, st>>>((const __nv_bfloat16*)proj, ld, taps_w, ring, chunk_seq, cu_chunk, cu, start, slots,
+                                                               A_log, dt_bias, z, z_ld, blocks, vblocks, s);
   const cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
 }
@@ -554,36 +713,43 @@ extern "C" int inv_conv_tail(const void* proj, int ld, int proj_f32, float* ring
   return e == cudaSuccess ? 0 : -(int)e;
 }
 
-// The recurrence over packed tokens: qn, kn [T, Hk, D], vv [T, H, Dv], g [T, g_ld], beta [T, H] -> o [T, H, Dv]; the state
-// [slots, H, D, Dv] is taken as zero for sequences with start = 0. g_ld and D are multiples of 4 or D is not.
-extern "C" int inv_delta_scan(const float* qn, const float* kn, const float* vv, const float* g, int g_ld, const float* beta, float* o, float* state,
-                              const int* cu, const int* start, const int* slots, int n_seq, const int* shape, void* stream) {
+// The recurrence over the chunks of n_seq sequences (blocks and vblocks of inv_delta_chunk) -> o [T, H, Dv]; the state
+// [slots, H, D, Dv] is taken as zero for sequences with start = 0.
+extern "C" int inv_delta_scan(const float* blocks, const float* vblocks, float* o, float* state, const int* cu_chunk, const int* cu, const int* start,
+                              const int* slots, int n_seq, int* status, const int* shape, void* stream) {
   const DeltaShape s = *reinterpret_cast<const DeltaShape*>(shape);
-  if (!delta_shape_ok(s) || (s.D % 4 == 0 && g_ld % 4)) return -ERR_BAD_ARG;
+  if (!delta_shape_ok(s)) return -ERR_BAD_ARG;
   if (n_seq <= 0) return 0;
-  cudaStream_t st = (cudaStream_t)stream;
-#define INV_SCAN(DP, LP, TH) launch_scan<DP, LP, TH>(qn, kn, vv, g, g_ld, beta, o, state, cu, start, slots, n_seq, s, st)
-  if (s.D <= 16) return INV_SCAN(16, 4, 64);
-  if (s.D <= 32) return INV_SCAN(32, 4, 64);
-  if (s.D <= 64) return INV_SCAN(64, 4, 64);
-  if (s.D <= 128) return INV_SCAN(128, 4, 64);
-  return INV_SCAN(256, 8, 64);
-#undef INV_SCAN
+  const int D4 = (s.D + 3) & ~3;
+  const int smem = (D4 * SC_COLS + 4 * 32 * SC_COLS + 2 * CH * SC_COLS + 2 * (block_floats(D4) + CH * SC_COLS)) * 4;
+  static bool configured = false;
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+    if (e != cudaSuccess) return -(int)e;
+    configured = true;
+  }
+  delta_scan_kernel<<<dim3((s.Dv + SC_COLS - 1) / SC_COLS, s.H, n_seq), SC_THREADS, smem, (cudaStream_t)stream>>>(blocks, vblocks, o, state, cu_chunk, cu,
+                                                                                                           start, slots, s.H, s.D, s.Dv, status);
+  const cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : -(int)e;
 }
 
 extern "C" int inv_gated_head_norm(const float* o, const float* w, const void* gate, int gate_ld, int gate_f32, void* out, int out_ld, int out_f32,
                                    int T, int H, int Dv, float eps, void* stream) {
   if (T <= 0) return 0;
-  const dim3 grid(T, (H + 3) / 4);
+  const long n_rows = (long)T * H;
+  const int grid = (int)((n_rows + 7) / 8);
+  const bool v4 = Dv % 4 == 0 && Dv <= 256 && gate_ld % 4 == 0 && out_ld % 4 == 0;
   cudaStream_t st = (cudaStream_t)stream;
-  if (gate_f32 && out_f32)
-    gated_head_norm_kernel<float, float><<<grid, 128, 0, st>>>(o, w, (const float*)gate, gate_ld, (float*)out, out_ld, H, Dv, eps);
-  else if (gate_f32)
-    gated_head_norm_kernel<float, __nv_bfloat16><<<grid, 128, 0, st>>>(o, w, (const float*)gate, gate_ld, (__nv_bfloat16*)out, out_ld, H, Dv, eps);
-  else if (!out_f32)
-    gated_head_norm_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, 128, 0, st>>>(o, w, (const __nv_bfloat16*)gate, gate_ld, (__nv_bfloat16*)out, out_ld,
-                                                                               H, Dv, eps);
+#define INV_HN(TG, TO)                                                                                                                          \
+  do {                                                                                                                                          \
+    if (v4) gated_head_norm_kernel<TG, TO, 4><<<grid, 256, 0, st>>>(o, w, (const TG*)gate, gate_ld, (TO*)out, out_ld, H, Dv, eps, n_rows);       \
+    else gated_head_norm_kernel<TG, TO, 1><<<grid, 256, 0, st>>>(o, w, (const TG*)gate, gate_ld, (TO*)out, out_ld, H, Dv, eps, n_rows);          \
+  } while (0)
+  if (gate_f32 && out_f32) INV_HN(float, float);
+  else if (!gate_f32 && !out_f32) INV_HN(__nv_bfloat16, __nv_bfloat16);
   else return -ERR_BAD_ARG;
+#undef INV_HN
   const cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
 }

@@ -14,6 +14,7 @@ from typing import List, Optional, Sequence
 
 import torch
 
+from ..ops.delta_rule import CHUNK
 from .kv_cache import PAGE, PagedRows
 
 
@@ -44,19 +45,25 @@ class StepBatch:
             want = [c - 1 for c in cu[1:]]
         self.n_want = len(want)
         self.want_all = list(want) == list(range(self.T))
-        self._buf = torch.empty(4 * self.n + 1 + 3 * self.T + self.n_want, dtype=torch.int32, device=self.device)
+        self.n_chunks = sum(-(-n // CHUNK) for n in lens)      # the delta rule advances chunk by chunk inside a portion
+        self._buf = torch.empty(5 * self.n + 2 + 3 * self.T + self.n_chunks + self.n_want, dtype=torch.int32, device=self.device)
         self._views()
         self._fill(cache, flat, cu, want)
 
     def _views(self):
-        sizes = [self.n, self.n, self.n, self.n + 1, self.T, self.T, self.T, self.n_want]
-        self.start, self.rows, self.slots, self.cu, self.ids, self.tok_seq, self.tok_pos, self.want = torch.split(self._buf[:sum(sizes)], sizes)
+        sizes = [self.n, self.n, self.n, self.n + 1, self.n + 1, self.n_chunks, self.T, self.T, self.T, self.n_want]
+        (self.start, self.rows, self.slots, self.cu, self.cu_chunk, self.chunk_seq, self.ids, self.tok_seq, self.tok_pos,
+         self.want) = torch.split(self._buf[:sum(sizes)], sizes)
 
     def _fill(self, cache, flat, cu, want):
         seq = [i for i, n in enumerate(self.lens) for _ in range(n)]
         pos = [s + k for s, n in zip(self.host_start, self.lens) for k in range(n)]
         slots = [cache.slot_of(r) for r in self.host_rows]
-        host = torch.tensor(self.host_start + self.host_rows + slots + cu + flat + seq + pos + list(want), dtype=torch.int32)
+        cu_chunk = [0]
+        for n in self.lens:
+            cu_chunk.append(cu_chunk[-1] - (-n // CHUNK))
+        chunk_seq = [i for i, n in enumerate(self.lens) for _ in range(-(-n // CHUNK))]
+        host = torch.tensor(self.host_start + self.host_rows + slots + cu + cu_chunk + chunk_seq + flat + seq + pos + list(want), dtype=torch.int32)
         self._buf[: host.numel()].copy_(host)
 
     def refill(self, cache, tokens: Sequence[int], start: Sequence[int], rows: Sequence[int]):

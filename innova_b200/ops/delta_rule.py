@@ -20,14 +20,16 @@ from . import runtime as rt
 
 _vp, _i, _f = _native.vp, _native.i32, _native.f32
 _native.register_cuda_sigs({
-    "inv_delta_prep": [_vp, _i, _i] + [_vp] * 12 + [_i, _vp, _i, _vp, _vp],
+    "inv_delta_chunk": [_vp, _i, _i] + [_vp] * 10 + [_i, _vp, _vp, _i, _vp, _vp],
     "inv_conv_tail": [_vp, _i, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp],
-    "inv_delta_scan": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp],
+    "inv_delta_scan": [_vp] * 8 + [_i, _vp, _vp, _vp],
     "inv_gated_head_norm": [_vp, _vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _i, _f, _vp],
     "inv_delta_decode": [_vp, _i, _i] + [_vp] * 8 + [_i, _vp, _i, _i, _vp, _f, _vp, _i, _i, _vp, _vp, _vp],
 })
 
-DECODE_MAX_TILE = 200 * 1024      # largest [D, Dv] fp32 state tile the one-launch decode kernel keeps in shared memory
+DECODE_MAX_TILE = 192 * 1024      # largest [D, Dv] fp32 state tile the one-launch decode kernel keeps in shared memory
+
+CHUNK = 16                         # tokens the prompt path advances per step of the recurrence
 
 
 def _pad8(n: int) -> int:
@@ -64,6 +66,12 @@ class DeltaShape:
     def tile_bytes(self) -> int:
         return self.D * self.Dv * 4
 
+    @property
+    def block_floats(self) -> int:
+        """Size of one (chunk, head) block between the chunk kernel and the scan (csrc/delta_rule.cu)."""
+        d4 = (self.D + 3) // 4 * 4
+        return 32 * d4 + CHUNK * d4 + CHUNK * 32 + d4
+
     def c_array(self):
         o = self.offsets
         return (C.c_int * 14)(self.H, self.Hk, self.D, self.Dv, self.taps, o[0], o[1], o[2], o[3], o[4], o[5], o[3], self.rank_a, self.rank_g)
@@ -71,25 +79,23 @@ class DeltaShape:
 
 def delta_prompt(s: DeltaShape, proj, z, gate, taps_w, A_log, dt_bias, norm_w, eps, ring, state, batch) -> torch.Tensor:
     """Packed tokens of several sequences -> normed, gated outputs [T, H * Dv] (type of ``gate``). ``z`` [T, >= H * D] fp32 is the
-    low-rank product of the decay (overwritten), ``gate`` [T, >= H * Dv] that of the output gate. Advances ``ring`` and ``state``."""
+    low-rank product of the decay, ``gate`` [T, >= H * Dv] that of the output gate. Advances ``ring`` and ``state``."""
     T = proj.shape[0]
     if not proj.is_cuda:
         return _delta_prompt_cpu(s, proj, z, gate, taps_w, A_log, dt_bias, norm_w, eps, ring, state, batch)
     dev, lib, st, arr = proj.device, rt.lib(), rt.stream_ptr(), s.c_array()
     pf = int(proj.dtype == torch.float32)
-    qn = torch.empty(T, s.Hk * s.D, dtype=torch.float32, device=dev)
-    kn = torch.empty_like(qn)
-    vv = torch.empty(T, s.H * s.Dv, dtype=torch.float32, device=dev)
-    beta = torch.empty(T, s.H, dtype=torch.float32, device=dev)
-    rt.check(lib.inv_delta_prep(proj.data_ptr(), proj.stride(0), pf, taps_w.data_ptr(), ring.data_ptr(), batch.tok_seq.data_ptr(),
-                                batch.tok_pos.data_ptr(), batch.start.data_ptr(), batch.slots.data_ptr(), A_log.data_ptr(), dt_bias.data_ptr(),
-                                qn.data_ptr(), kn.data_ptr(), vv.data_ptr(), z.data_ptr(), z.stride(0), beta.data_ptr(), T, arr, st), "inv_delta_prep")
+    blocks = torch.empty(batch.n_chunks * s.H * s.block_floats, dtype=torch.float32, device=dev)
+    vblocks = torch.empty(batch.n_chunks * s.H * ((s.Dv + 15) // 16) * 256, dtype=torch.float32, device=dev)
+    rt.check(lib.inv_delta_chunk(proj.data_ptr(), proj.stride(0), pf, taps_w.data_ptr(), ring.data_ptr(), batch.chunk_seq.data_ptr(),
+                                 batch.cu_chunk.data_ptr(), batch.cu.data_ptr(), batch.start.data_ptr(), batch.slots.data_ptr(), A_log.data_ptr(),
+                                 dt_bias.data_ptr(), z.data_ptr(), z.stride(0), blocks.data_ptr(), vblocks.data_ptr(), batch.n_chunks, arr, st),
+             "inv_delta_chunk")
     rt.check(lib.inv_conv_tail(proj.data_ptr(), proj.stride(0), pf, ring.data_ptr(), batch.cu.data_ptr(), batch.start.data_ptr(),
                                batch.slots.data_ptr(), batch.n, arr, st), "inv_conv_tail")
     o = torch.empty(T, s.H * s.Dv, dtype=torch.float32, device=dev)
-    rt.check(lib.inv_delta_scan(qn.data_ptr(), kn.data_ptr(), vv.data_ptr(), z.data_ptr(), z.stride(0), beta.data_ptr(), o.data_ptr(),
-                                state.data_ptr(), batch.cu.data_ptr(), batch.start.data_ptr(), batch.slots.data_ptr(), batch.n, arr, st),
-             "inv_delta_scan")
+    rt.check(lib.inv_delta_scan(blocks.data_ptr(), vblocks.data_ptr(), o.data_ptr(), state.data_ptr(), batch.cu_chunk.data_ptr(), batch.cu.data_ptr(),
+                                batch.start.data_ptr(), batch.slots.data_ptr(), batch.n, rt.status_tensor(dev).data_ptr(), arr, st), "inv_delta_scan")
     from .hyper import row_buffer
     out = row_buffer(T, s.H * s.Dv, gate.dtype, dev)
     f32 = int(gate.dtype == torch.float32)
