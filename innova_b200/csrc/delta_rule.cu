@@ -46,7 +46,7 @@ struct DeltaShape {
 };
 
 constexpr int CH = 16;         // tokens per chunk
-constexpr int CH_TAPS = 8;     // longest convolution kept in registers while a thread walks down a chunk
+constexpr int CK_THREADS = 128;
 
 // One (chunk, head) block of floats: decayed keys and queries [D4][16 k | 16 q], keys for the update [16][D4], the maps
 // [16 s][16 T | 16 PT], the chunk's decay [D4]; D4 = D rounded up to 4.
@@ -60,14 +60,27 @@ __device__ __forceinline__ float conv_in(const T* proj, int ld, const float* rin
 }
 
 // ------------------------------------------------------------------------------------------------ prompt: chunks
-template <typename T>
-__global__ void __launch_bounds__(256) delta_chunk_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ taps_w,
-                                                          const float* __restrict__ ring0, const int* __restrict__ chunk_seq,
-                                                          const int* __restrict__ cu_chunk, const int* __restrict__ cu,
-                                                          const int* __restrict__ start_, const int* __restrict__ slots,
-                                                          const float* __restrict__ A_log, const float* __restrict__ dt_bias,
-                                                          const float* __restrict__ z, int z_ld, float* __restrict__ blocks,
-                                                          float* __restrict__ vblocks, const DeltaShape s) {
+// One exchange of the sums over 16 lanes: 2 M values per lane become M, and so on down to two.
+template <int M>
+__device__ __forceinline__ void fold_lanes(float* v, int l) {
+  const bool up = (l & (M / 2)) != 0;
+#pragma unroll
+  for (int j = 0; j < M; ++j) {
+    const float give = up ? v[j] : v[j + M], keep = up ? v[j + M] : v[j];
+    v[j] = keep + __shfl_xor_sync(0xffffffffu, give, M / 2);
+  }
+  if constexpr (M > 2) fold_lanes<M / 2>(v, l);
+}
+
+// TAPS: longest convolution a thread keeps in registers while it walks down the chunk (longer ones re-read their inputs).
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(CK_THREADS, 6) delta_chunk_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ taps_w,
+                                                                    const float* __restrict__ ring0, const int* __restrict__ chunk_seq,
+                                                                    const int* __restrict__ cu_chunk, const int* __restrict__ cu,
+                                                                    const int* __restrict__ start_, const int* __restrict__ slots,
+                                                                    const float* __restrict__ A_log, const float* __restrict__ dt_bias,
+                                                                    const float* __restrict__ z, int z_ld, float* __restrict__ blocks,
+                                                                    float* __restrict__ vblocks, const DeltaShape s) {
   extern __shared__ __align__(16) float csm[];
   __shared__ float kap[CH][CH + 4], P[CH][CH + 4], Tm[CH][CH + 4], beta[CH];
   const int D = s.D, Dv = s.Dv, D4 = (D + 3) & ~3, cgs = (Dv + 15) / 16;
@@ -81,48 +94,63 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(const T* __restrict__ 
   const float* ring = ring0 + (size_t)slots[seq] * s.taps * s.channels;
   float* blk = blocks + ((size_t)ch * s.H + h) * block_floats(D4);
   float* vb = vblocks + ((size_t)ch * s.H + h) * cgs * (CH * 16);
-  for (int i = tid; i < 2 * D + cgs * 16; i += 256) {
-    const int v = i - 2 * D;
+  // a thread convolves one channel over half the chunk
+  constexpr int HALF = CH / 2;
+  const int n_ch = 2 * D + cgs * 16;
+  for (int j = tid; j < 2 * n_ch; j += CK_THREADS) {
+    const int half = j >= n_ch, i = half ? j - n_ch : j, v = i - 2 * D, tb = half * HALF;
+    float* dst = i < D ? q_s + i : i < 2 * D ? k_s + (i - D) : vb + (size_t)(v >> 4) * (CH * 16) + (v & 15);
+    const int step = i < 2 * D ? D : 16;
     if (v >= Dv) {                                 // padding columns of the last group
-      for (int t = 0; t < CH; ++t) vb[(size_t)(v >> 4) * (CH * 16) + t * 16 + (v & 15)] = 0.f;
+      for (int t = tb; t < tb + HALF; ++t) dst[t * step] = 0.f;
       continue;
     }
     const int c = i < D ? s.off_q + hk * D + i : i < 2 * D ? s.off_k + hk * D + (i - D) : s.off_v + h * Dv + v;
-    float win[CH_TAPS], w[CH_TAPS];                // win[j]: input j + 1 tokens back
-    const bool slide = s.taps <= CH_TAPS;
+    const T* col = proj + (row0 + c0) * ld + c;
+    if (s.taps <= TAPS) {
+      float in[HALF + TAPS - 1], w[TAPS];          // inputs tb - (TAPS - 1) .. tb + HALF - 1
 #pragma unroll
-    for (int j = 0; j < CH_TAPS; ++j) {
-      w[j] = j < s.taps ? taps_w[(size_t)(s.taps - 1 - j) * s.channels + c] : 0.f;
-      win[j] = j + 1 < s.taps ? conv_in(proj, ld, ring, s, row0, start, pos0 - 1 - j, c) : 0.f;
-    }
+      for (int k = 0; k < TAPS; ++k) w[k] = k < s.taps ? taps_w[(size_t)(s.taps - 1 - k) * s.channels + c] : 0.f;
 #pragma unroll
-    for (int t = 0; t < CH; ++t) {
-      const float x = t < n ? dr_ld(proj + (row0 + c0 + t) * ld + c) : 0.f;
-      float a = x * w[0];
-      if (slide) {
-#pragma unroll
-        for (int j = 1; j < CH_TAPS; ++j) a = fmaf(win[j - 1], w[j], a);
-      } else {
-        for (int j = 1; j < s.taps; ++j)
-          a = fmaf(conv_in(proj, ld, ring, s, row0, start, pos0 + t - j, c), taps_w[(size_t)(s.taps - 1 - j) * s.channels + c], a);
+      for (int k = 0; k < TAPS - 1; ++k) {
+        const int t = tb + k - (TAPS - 1);
+        in[k] = TAPS - 1 - k < s.taps ? conv_in(proj, ld, ring, s, row0, start, pos0 + t, c) : 0.f;
       }
 #pragma unroll
-      for (int j = CH_TAPS - 1; j > 0; --j) win[j] = win[j - 1];
-      win[0] = x;
-      a = t < n ? dr_silu(a) : 0.f;
-      if (i < D) q_s[t * D + i] = a;
-      else if (i < 2 * D) k_s[t * D + i - D] = a;
-      else vb[(size_t)(v >> 4) * (CH * 16) + t * 16 + (v & 15)] = a;
+      for (int k = 0; k < HALF; ++k) in[TAPS - 1 + k] = tb + k < n ? dr_ld(col + (long)(tb + k) * ld) : 0.f;
+#pragma unroll
+      for (int k = 0; k < HALF; ++k) {
+        float a = 0.f;
+#pragma unroll
+        for (int m = 0; m < TAPS; ++m) a = fmaf(in[TAPS - 1 + k - m], w[m], a);
+        dst[(tb + k) * step] = tb + k < n ? dr_silu(a) : 0.f;
+      }
+    } else {
+      for (int t = tb; t < tb + HALF; ++t) {
+        float a = 0.f;
+        if (t < n)
+          for (int m = 0; m < s.taps; ++m)
+            a = fmaf(conv_in(proj, ld, ring, s, row0, start, pos0 + t - m, c), taps_w[(size_t)(s.taps - 1 - m) * s.channels + c], a);
+        dst[t * step] = dr_silu(a);
+      }
     }
   }
   const float ea = expf(A_log[h]);
-  for (int i = tid; i < CH * D; i += 256) {
-    const int t = i / D, d = i % D;
-    g_s[i] = t < n ? expf(-ea * dr_softplus(z[(row0 + c0 + t) * z_ld + h * D + d] + dt_bias[h * D + d])) : 1.f;
+  for (int d = tid; d < D; d += CK_THREADS) {
+    const float bias = dt_bias[h * D + d];
+    const float* zp = z + (row0 + c0) * z_ld + h * D + d;
+#pragma unroll
+    for (int t0 = 0; t0 < CH; t0 += 8) {
+      float x[8];
+#pragma unroll
+      for (int t = 0; t < 8; ++t) x[t] = t0 + t < n ? zp[(long)(t0 + t) * z_ld] : 0.f;
+#pragma unroll
+      for (int t = 0; t < 8; ++t) g_s[(t0 + t) * D + d] = t0 + t < n ? expf(-ea * dr_softplus(x[t] + bias)) : 1.f;
+    }
   }
   if (tid < CH) beta[tid] = tid < n ? dr_sigmoid(dr_ld(proj + (row0 + c0 + tid) * ld + s.off_b + h)) : 0.f;
   __syncthreads();
-  for (int t = warp; t < CH; t += 8) {             // unit vectors; the query also carries D^-1/2
+  for (int t = warp; t < CH; t += CK_THREADS / 32) {   // unit vectors; the query also carries D^-1/2
     float sq = 0.f, sk = 0.f;
     for (int d = lane; d < D; d += 32) {
       sq = fmaf(q_s[t * D + d], q_s[t * D + d], sq);
@@ -136,57 +164,66 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(const T* __restrict__ 
   }
   __syncthreads();
   // decayed keys and queries, and the keys of the update: a running product down the chunk and one up
-  for (int d = tid; d < D4; d += 256) {
-    float kq[2][CH], G = 1.f;
-    if (d < D) {
+  for (int d = tid; d < D4; d += CK_THREADS) {
+    const bool in = d < D;
+    float G = 1.f;
 #pragma unroll
-      for (int t = 0; t < CH; ++t) {
-        G *= g_s[t * D + d];
-        kq[0][t] = k_s[t * D + d] * G;
-        kq[1][t] = q_s[t * D + d] * G;
+    for (int t = 0; t < CH; t += 4) {
+      float kk[4], qq[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        if (in) G *= g_s[(t + j) * D + d];
+        kk[j] = in ? k_s[(t + j) * D + d] * G : 0.f;
+        qq[j] = in ? q_s[(t + j) * D + d] * G : 0.f;
       }
-    } else {
-#pragma unroll
-      for (int t = 0; t < CH; ++t) kq[0][t] = kq[1][t] = 0.f;
+      *reinterpret_cast<float4*>(blk + (size_t)d * 32 + t) = make_float4(kk[0], kk[1], kk[2], kk[3]);
+      *reinterpret_cast<float4*>(blk + (size_t)d * 32 + CH + t) = make_float4(qq[0], qq[1], qq[2], qq[3]);
     }
-#pragma unroll
-    for (int t = 0; t < 2 * CH; t += 4)
-      *reinterpret_cast<float4*>(blk + (size_t)d * 32 + t) =
-          make_float4(kq[t / CH][t % CH], kq[t / CH][t % CH + 1], kq[t / CH][t % CH + 2], kq[t / CH][t % CH + 3]);
     blk[32 * D4 + CH * D4 + CH * 32 + d] = G;
     float R = 1.f;
 #pragma unroll
     for (int t = CH - 1; t >= 0; --t) {
-      blk[32 * D4 + t * D4 + d] = d < D ? k_s[t * D + d] * R : 0.f;
-      if (d < D) R *= g_s[t * D + d];
+      blk[32 * D4 + t * D4 + d] = in ? k_s[t * D + d] * R : 0.f;
+      if (in) R *= g_s[t * D + d];
     }
   }
-  // kap and P: 16 lanes per source token s share the channels and walk t upwards with w = k_s * (decays of s + 1 .. t)
+  // kap and P: 16 lanes per source token share the channels and walk upwards with w = k_src * (decays of src + 1 .. t). A warp
+  // takes sources 2 m and 2 m + 1 (about the same length) for m = warp and 7 - warp, which evens out the warps.
   {
-    const int src = tid >> 4, l = tid & 15;
-    float ak[CH], ap[CH];
+    const int l = lane & 15;
 #pragma unroll
-    for (int t = 0; t < CH; ++t) ak[t] = ap[t] = 0.f;
-    for (int d = l; d < D; d += 16) {
-      float w = k_s[src * D + d];
+    for (int pass = 0; pass < 2; ++pass) {
+      const int src = 2 * (pass ? 7 - warp : warp) + (lane >> 4), steps = CH - src;
+      float v[2 * CH];                             // [j] kap, [16 + j] P for t = src + j
 #pragma unroll
-      for (int t = 0; t < CH; ++t)
-        if (t >= src) {
-          if (t > src) w *= g_s[t * D + d];
-          ak[t] = fmaf(k_s[t * D + d], w, ak[t]);
-          ap[t] = fmaf(q_s[t * D + d], w, ap[t]);
+      for (int j = 0; j < 2 * CH; ++j) v[j] = 0.f;
+      for (int d = l; d < D; d += 16) {
+        const float* kp = k_s + src * D + d;
+        const float* qp = q_s + src * D + d;
+        const float* gp = g_s + src * D + d;
+        float w = kp[0];
+#pragma unroll
+        for (int j = 0; j < CH; ++j) {
+          if (j < steps) {
+            if (j > 0) w *= gp[j * D];
+            v[j] = fmaf(kp[j * D], w, v[j]);
+            v[CH + j] = fmaf(qp[j * D], w, v[CH + j]);
+          }
         }
-    }
-#pragma unroll
-    for (int t = 0; t < CH; ++t) {
-#pragma unroll
-      for (int o = 8; o > 0; o >>= 1) {
-        ak[t] += __shfl_xor_sync(0xffffffffu, ak[t], o);
-        ap[t] += __shfl_xor_sync(0xffffffffu, ap[t], o);
       }
-      if (l == 0) {
-        kap[t][src] = t > src ? ak[t] : 0.f;
-        P[t][src] = t >= src ? ap[t] : 0.f;
+      // sums over the 16 lanes: each exchange halves the values a lane is responsible for; lane l ends with v[2 l'], v[2 l' + 1]
+      fold_lanes<CH>(v, l);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int j = 2 * (l & 7) + e, t = src + j;
+        if (t < CH) {
+          if (l < 8) kap[t][src] = j > 0 ? v[e] : 0.f;
+          else P[t][src] = v[e];
+        }
+        if (j < src) {                             // targets before the source
+          if (l < 8) kap[j][src] = 0.f;
+          else P[j][src] = 0.f;
+        }
       }
     }
   }
@@ -195,17 +232,19 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(const T* __restrict__ 
     float x[CH];
 #pragma unroll
     for (int t = 0; t < CH; ++t) {
-      float a = t == tid ? 1.f : 0.f;
+      float a = t == tid ? 1.f : 0.f, a2 = 0.f;
 #pragma unroll
-      for (int r = 0; r < CH; ++r)
+      for (int r = 0; r < CH; r += 2) {
         if (r < t) a = fmaf(-kap[t][r], x[r], a);
-      x[t] = beta[t] * a;
+        if (r + 1 < t) a2 = fmaf(-kap[t][r + 1], x[r + 1], a2);
+      }
+      x[t] = beta[t] * (a + a2);
       Tm[t][tid] = x[t];
     }
   }
   __syncthreads();
-  {
-    const int t = tid & 15, c = tid >> 4;          // entry (t, c) of T and of P T
+  for (int i = tid; i < CH * CH; i += CK_THREADS) {
+    const int t = i & 15, c = i >> 4;              // entry (t, c) of T and of P T
     float a = 0.f;
 #pragma unroll
     for (int r = 0; r < CH; ++r) a = fmaf(P[t][r], Tm[r][c], a);
@@ -436,10 +475,25 @@ __global__ void __launch_bounds__(256) gated_head_norm_kernel(const float* __res
 // memory while the convolutions, norms and low-rank products run, it is updated in place and a bulk copy writes it back.
 // Row groups of threads walk the tile (VEC value columns per thread); three tiles of 128 x 128 share an SM.
 constexpr int DD_THREADS = 256;
+
+// a[j] += f * (element j of a 16-byte piece)
+__device__ __forceinline__ void fma_row(const uint4& p, float f, float* a, __nv_bfloat16) {
+  const uint32_t u[4] = {p.x, p.y, p.z, p.w};
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    a[2 * j] = fmaf(__uint_as_float(u[j] << 16), f, a[2 * j]);
+    a[2 * j + 1] = fmaf(__uint_as_float(u[j] & 0xffff0000u), f, a[2 * j + 1]);
+  }
+}
+__device__ __forceinline__ void fma_row(const uint4& p, float f, float* a, float) {
+  a[0] = fmaf(__uint_as_float(p.x), f, a[0]); a[1] = fmaf(__uint_as_float(p.y), f, a[1]);
+  a[2] = fmaf(__uint_as_float(p.z), f, a[2]); a[3] = fmaf(__uint_as_float(p.w), f, a[3]);
+}
+
 constexpr int DD_MAX_TILE = 192 * 1024;
 
 template <typename T, typename TW, typename TO, int VEC>
-__global__ void __launch_bounds__(DD_THREADS) delta_decode_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ taps_w,
+__global__ void __launch_bounds__(DD_THREADS, 3) delta_decode_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ taps_w,
                                                                   float* __restrict__ ring0, float* __restrict__ state0,
                                                                   const int* __restrict__ pos_, const int* __restrict__ slots,
                                                                   const float* __restrict__ A_log, const float* __restrict__ dt_bias,
@@ -480,6 +534,22 @@ __global__ void __launch_bounds__(DD_THREADS) delta_decode_kernel(const T* __res
                    : "memory");
     }
   }
+  // everything later phases read from global memory is requested here, so that the waits overlap: small vectors, and this
+  // thread's first rows of the low-rank matrices
+  constexpr int VW = 16 / sizeof(TW), PRE = 8;
+  const int dg = (D + VW - 1) / VW, vg = (Dv + VW - 1) / VW;
+  const bool vec = D % VW == 0 && Dv % VW == 0;   // rows are 16-byte multiples, so every piece is aligned
+  const bool pre_a = lane < dg;
+  const int pre_c = (pre_a ? lane : lane - dg) * VW, pre_rank = pre_a ? s.rank_a : s.rank_g;
+  const TW* pre_w = (pre_a ? a2t + h * D : g2t + h * Dv) + pre_c;
+  const int pre_ld = pre_a ? a2_ld : g2_ld;
+  uint4 pre[PRE];
+#pragma unroll
+  for (int i = 0; i < PRE; ++i) {
+    const int r = warp + i * NW;
+    pre[i] = (vec && lane < dg + vg && r < pre_rank) ? *reinterpret_cast<const uint4*>(pre_w + (size_t)r * pre_ld) : make_uint4(0, 0, 0, 0);
+  }
+  const float a_log = A_log[h], b_in = dr_ld(row + s.off_b + h), bias0 = tid < D ? dt_bias[h * D + tid] : 0.f, nw0 = tid < Dv ? norm_w[tid] : 0.f;
   if (pos == 0)
     for (int i = tid; i < D * Dv; i += DD_THREADS) S[i] = 0.f;
   else if (!bulk)
@@ -488,12 +558,25 @@ __global__ void __launch_bounds__(DD_THREADS) delta_decode_kernel(const T* __res
   const int nq = 2 * D + Dv;
   const bool own_qk = h % (s.H / s.Hk) == 0;
   float ssq = 0.f, ssk = 0.f;
+#pragma unroll 2
   for (int i = tid; i < nq; i += DD_THREADS) {
     const int c = i < D ? s.off_q + hk * D + i : i < 2 * D ? s.off_k + hk * D + (i - D) : s.off_v + h * Dv + (i - 2 * D);
     const float cur = dr_ld(row + c);
     float a = cur * taps_w[(size_t)(s.taps - 1) * s.channels + c];
-    for (int j = 1; j < s.taps; ++j)
-      if (pos - j >= 0) a = fmaf(ring[(size_t)((pos - j) % s.taps) * s.channels + c], taps_w[(size_t)(s.taps - 1 - j) * s.channels + c], a);
+    if (s.taps <= 4) {
+      float x[3], w[3];
+#pragma unroll
+      for (int j = 1; j < 4; ++j) {
+        const bool in = j < s.taps && pos - j >= 0;
+        x[j - 1] = in ? ring[(size_t)((pos - j) % s.taps) * s.channels + c] : 0.f;
+        w[j - 1] = in ? taps_w[(size_t)(s.taps - 1 - j) * s.channels + c] : 0.f;
+      }
+#pragma unroll
+      for (int j = 0; j < 3; ++j) a = fmaf(x[j], w[j], a);
+    } else {
+      for (int j = 1; j < s.taps; ++j)
+        if (pos - j >= 0) a = fmaf(ring[(size_t)((pos - j) % s.taps) * s.channels + c], taps_w[(size_t)(s.taps - 1 - j) * s.channels + c], a);
+    }
     if (i >= 2 * D || own_qk) ring[(size_t)(pos % s.taps) * s.channels + c] = cur;
     a = dr_silu(a);
     if (i < D) { q_s[i] = a; ssq = fmaf(a, a, ssq); }
@@ -510,39 +593,39 @@ __global__ void __launch_bounds__(DD_THREADS) delta_decode_kernel(const T* __res
   const float rq = 1.0f / sqrtf(nq2 + 1e-6f) * (1.0f / sqrtf((float)D)), rk = 1.0f / sqrtf(nk2 + 1e-6f);
   // low-rank decay and output gate (their second matrices are stored transposed: [rank, heads * channels]): a thread adds VW
   // neighbouring channels over every eighth rank row, and the eight partial sums meet in shared memory
-  const float ea = expf(A_log[h]);
-  {
-    constexpr int VW = 16 / sizeof(TW);
-    const int dg = (D + VW - 1) / VW, vg = (Dv + VW - 1) / VW;
-    const bool vec = D % VW == 0 && Dv % VW == 0;   // rows are 16-byte multiples, so every piece is aligned
-    for (int p = lane; p < dg + vg; p += 32) {
-      const bool is_a = p < dg;
-      const int c = (is_a ? p : p - dg) * VW, width = is_a ? D : Dv, rank = is_a ? s.rank_a : s.rank_g, ldw = is_a ? a2_ld : g2_ld;
-      const TW* w = (is_a ? a2t + h * D : g2t + h * Dv) + c;
-      const float* f = lr + (is_a ? 0 : s.rank_a);
-      float a[VW];
+  const float ea = expf(a_log);
+  for (int p = lane; p < dg + vg; p += 32) {
+    const bool is_a = p < dg;
+    const int c = (is_a ? p : p - dg) * VW, width = is_a ? D : Dv, rank = is_a ? s.rank_a : s.rank_g, ldw = is_a ? a2_ld : g2_ld;
+    const TW* w = (is_a ? a2t + h * D : g2t + h * Dv) + c;
+    const float* f = lr + (is_a ? 0 : s.rank_a);
+    float a[VW];
 #pragma unroll
-      for (int j = 0; j < VW; ++j) a[j] = 0.f;
-      if (vec) {
-#pragma unroll 8
-        for (int r = warp; r < rank; r += NW) {
-          float x[VW];
+    for (int j = 0; j < VW; ++j) a[j] = 0.f;
+    int r0 = warp;
+    if (vec) {
+      if (p == lane) {                             // the rows requested at the start
 #pragma unroll
-          for (int j = 0; j < VW; j += 4) dr_ld4(w + (size_t)r * ldw + j, x + j);
-          const float fr = f[r];
-#pragma unroll
-          for (int j = 0; j < VW; ++j) a[j] = fmaf(x[j], fr, a[j]);
+        for (int i = 0; i < PRE; ++i) {
+          const float fr = warp + i * NW < rank ? f[warp + i * NW] : 0.f;
+          fma_row(pre[i], fr, a, TW());
         }
-      } else {
-        for (int r = warp; r < rank; r += NW)
-#pragma unroll
-          for (int j = 0; j < VW; ++j)
-            if (c + j < width) a[j] = fmaf(dr_ld(w + (size_t)r * ldw + j), f[r], a[j]);
+        r0 += PRE * NW;
       }
+#pragma unroll 8
+      for (int r = r0; r < rank; r += NW) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(w + (size_t)r * ldw);
+        fma_row(raw, f[r], a, TW());
+      }
+    } else {
+      for (int r = r0; r < rank; r += NW)
 #pragma unroll
-      for (int j = 0; j < VW; ++j)
-        if (c + j < width) low[warp * (D + Dv) + (is_a ? 0 : D) + c + j] = a[j];
+        for (int j = 0; j < VW; ++j)
+          if (c + j < width) a[j] = fmaf(dr_ld(w + (size_t)r * ldw + j), f[r], a[j]);
     }
+#pragma unroll
+    for (int j = 0; j < VW; ++j)
+      if (c + j < width) low[warp * (D + Dv) + (is_a ? 0 : D) + c + j] = a[j];
   }
   __syncthreads();
   for (int d = tid; d < D + Dv; d += DD_THREADS) {
@@ -550,14 +633,14 @@ __global__ void __launch_bounds__(DD_THREADS) delta_decode_kernel(const T* __res
 #pragma unroll
     for (int i = 0; i < NW; ++i) a += low[i * (D + Dv) + d];
     if (d < D) {
-      g_s[d] = expf(-ea * dr_softplus(a + dt_bias[h * D + d]));
+      g_s[d] = expf(-ea * dr_softplus(a + (d == tid ? bias0 : dt_bias[h * D + d])));
       q_s[d] *= rq;
       k_s[d] *= rk;
     } else {
       gate_s[d - D] = dr_sigmoid(a);
     }
   }
-  const float beta = dr_sigmoid(dr_ld(row + s.off_b + h));
+  const float beta = dr_sigmoid(b_in);
   bool ok = true;
   if (bulk && pos > 0) ok = mbar_wait(&bar, 0, &abort_flag, status, ERR_WAIT_FULL);
   if (!__syncthreads_and(ok)) {  // the copy never arrived: leave it a bounded time before the shared memory goes away
@@ -639,7 +722,7 @@ __global__ void __launch_bounds__(DD_THREADS) delta_decode_kernel(const T* __res
   if (tid < Dv) {
     float tot = 0.f;
     for (int i = 0; i < NW; ++i) tot += ws[i];
-    dr_st(out + (size_t)b * out_ld + h * Dv + tid, ov * (1.0f / sqrtf(tot / (float)Dv + eps)) * norm_w[tid] * gate_s[tid]);
+    dr_st(out + (size_t)b * out_ld + h * Dv + tid, ov * (1.0f / sqrtf(tot / (float)Dv + eps)) * nw0 * gate_s[tid]);
   }
   if (bulk && tid == 0) asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");
 }
@@ -683,19 +766,26 @@ extern "C" int inv_delta_chunk(const void* proj, int ld, int proj_f32, const flo
   const dim3 grid(n_chunks, s.H);
   const int smem = 3 * CH * s.D * 4;   // at most 48 KB
   cudaStream_t st = (cudaStream_t)stream;
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(delta_chunk_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 3 * CH * 256 * 4);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_chunk_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 3 * CH * 256 * 4);
-    if (e != cudaSuccess) return -(int)e;
-    configured = true;
+  // channels above 192 need more than the default 48 KB with the static arrays
+#define INV_CK(T, TAPS)                                                                                                                              \
+  do {                                                                                                                                               \
+    static bool configured = false;                                                                                                                  \
+    if (!configured) {                                                                                                                               \
+      const cudaError_t e = cudaFuncSetAttribute(delta_chunk_kernel<T, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 3 * CH * 256 * 4);         \
+      if (e != cudaSuccess) return -(int)e;                                                                                                          \
+      configured = true;                                                                                                                             \
+    }                                                                                                                                                \
+    delta_chunk_kernel<T, TAPS><<<grid, CK_THREADS, smem, st>>>((const T*)proj, ld, taps_w, ring, chunk_seq, cu_chunk, cu, start, slots, A_log, dt_bias, \
+                                                                z, z_ld, blocks, vblocks, s);                                                        \
+  } while (0)
+  if (proj_f32) {
+    if (s.taps <= 4) INV_CK(float, 4);
+    else INV_CK(float, 8);
+  } else {
+    if (s.taps <= 4) INV_CK(__nv_bfloat16, 4);
+    else INV_CK(__nv_bfloat16, 8);
   }
-  if (proj_f32)
-    delta_chunk_kernel<float><<<grid, 256, smem, st>>>((const float*)proj, ld, taps_w, ring, chunk_seq, cu_chunk, cu, start, slots, A_log, dt_bias, z,
-                                                       z_ld, blocks, vblocks, s);
-  else
-    delta_chunk_kernel<__nv_bfloat16><<<grid, 256, smem, st>>>((const __nv_bfloat16*)proj, ld, taps_w, ring, chunk_seq, cu_chunk, cu, start, slots,
-                                                               A_log, dt_bias, z, z_ld, blocks, vblocks, s);
+#undef INV_CK
   const cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
 }

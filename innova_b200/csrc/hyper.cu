@@ -82,9 +82,9 @@ __device__ __forceinline__ float hc_block_sum(float v, float* red) {
 
 // NS: number of streams at compile time, 0 = read from the parameters.
 template <int NS, typename YT, typename HT, int V>
-__global__ void __launch_bounds__(256) hyper_step_kernel(const HyperParams p) {
+__global__ void __launch_bounds__(NS > 0 ? 512 : 256) hyper_step_kernel(const HyperParams p) {
   extern __shared__ float hc_u[];  // [E]
-  __shared__ float red[8];
+  __shared__ float red[16];
   __shared__ float s_mix[HC_MAX_STREAMS * HC_MAX_STREAMS], s_out[HC_MAX_STREAMS], s_in[HC_MAX_STREAMS];
   constexpr int CAP = NS > 0 ? NS : HC_MAX_STREAMS;
   const int S = NS > 0 ? NS : p.S;
@@ -188,7 +188,8 @@ __global__ void __launch_bounds__(256) hyper_step_kernel(const HyperParams p) {
 template <typename YT, typename HT, int V>
 static int hyper_launch(const HyperParams& p, int n, cudaStream_t st) {
   int threads = ((p.E + V - 1) / V + 31) / 32 * 32;
-  if (threads > 256) threads = 256;
+  const int cap = n <= 148 ? 512 : 256;  // few rows: one pass over a row, its latency is all there is
+  if (threads > cap) threads = cap;
   const size_t smem = (size_t)p.E * 4;
   switch (p.S) {
     case 1: hyper_step_kernel<1, YT, HT, V><<<n, threads, smem, st>>>(p); break;

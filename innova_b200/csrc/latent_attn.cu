@@ -371,17 +371,26 @@ __global__ void __launch_bounds__(128) latent_attend_mma_kernel(const __nv_bfloa
   }
 }
 
+constexpr int LA_MAX_SPLITS = 32;
 __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ part, __nv_bfloat16* __restrict__ out, int Rp, int splits) {
+  __shared__ float wt[LA_MAX_SPLITS];
   const size_t th = blockIdx.x;
   const float* p = part + th * splits * (size_t)(Rp + 2);
-  float m = -INFINITY, l = 0.f;
-  for (int i = 0; i < splits; ++i) m = fmaxf(m, p[(size_t)i * (Rp + 2) + Rp]);
-  for (int i = 0; i < splits; ++i) l += p[(size_t)i * (Rp + 2) + Rp + 1] * exp2f(p[(size_t)i * (Rp + 2) + Rp] - m);
-  const float inv = 1.0f / l;
+  if (threadIdx.x < 32) {
+    const bool in = (int)threadIdx.x < splits;
+    const float m = in ? p[(size_t)threadIdx.x * (Rp + 2) + Rp] : -INFINITY, l = in ? p[(size_t)threadIdx.x * (Rp + 2) + Rp + 1] : 0.f;
+    float mx = m;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    const float e = exp2f(m - mx);
+    wt[threadIdx.x] = e / la_warp_sum(l * e);
+  }
+  __syncthreads();
   for (int c = threadIdx.x; c < Rp; c += 128) {
     float a = 0.f;
-    for (int i = 0; i < splits; ++i) a = fmaf(p[(size_t)i * (Rp + 2) + c], exp2f(p[(size_t)i * (Rp + 2) + Rp] - m), a);
-    out[th * Rp + c] = __float2bfloat16_rn(a * inv);
+#pragma unroll 8
+    for (int i = 0; i < splits; ++i) a = fmaf(p[(size_t)i * (Rp + 2) + c], wt[i], a);
+    out[th * Rp + c] = __float2bfloat16_rn(a);
   }
 }
 
@@ -477,7 +486,7 @@ extern "C" int inv_latent_attend(const void* q, const void* pool, int f32, int R
   if (f32) {
     rc = launch_attend<float>(q, pool, Rp, page_table, max_pages, rows, tok_seq, tok_pos, window, scale, out, T, H, st);
   } else {
-    if (Rp % 16 || splits < 1 || splits > 64 || (splits > 1 && !part)) return -ERR_BAD_ARG;
+    if (Rp % 16 || splits < 1 || splits > LA_MAX_SPLITS || (splits > 1 && !part)) return -ERR_BAD_ARG;
 #define INV_LM(NT) launch_mma<NT>(q, pool, Rp, page_table, max_pages, rows, tok_seq, tok_pos, window, scale, out, part, splits, T, H, st)
     if (Rp <= 64) rc = INV_LM(2);
     else if (Rp <= 128) rc = INV_LM(4);
