@@ -248,9 +248,8 @@ def kernel_section(size="2k"):
         report("paged_decode", f"B{B} H{H} D128 context {WINDOW}", cold(lambda: kv.decode_attention(0, qh, H, 0.09)), B * WINDOW * H * 128 * 4 / 1e9,
                tflop=B * H * WINDOW * 128 * 4 / 1e12, like="latent_attend")
         wl, xl = rand(4096, E).to(bf), rand(B, E).to(bf)
-        acc = torch.zeros(64, 4096, device=dev)
-        report("gemm split-K (decode projection)", f"M{B} N4096 K{E}", cold(lambda: ops.gemm(xl, wl, out=acc[:B], epilogue=ops.EPI_ATOMIC)), wl.numel() * 2 / 1e9)
-        report("gemm", f"M{B} N4096 K{E}", cold(lambda: ops.gemm(xl, wl)), wl.numel() * 2 / 1e9, like="gemm split-K (decode projection)")
+        report("skinny_gemm", f"M{B} N4096 K{E}", cold(lambda: ops.skinny_gemm(xl, wl)), wl.numel() * 2 / 1e9)
+        report("gemm", f"M{B} N4096 K{E}", cold(lambda: ops.gemm(xl, wl)), wl.numel() * 2 / 1e9, like="skinny_gemm")
     # attention, prompts
     T = 8192
     c = LatentStateCache([(R, WINDOW)], [], 1, T, dev)

@@ -516,7 +516,7 @@ __global__ void __launch_bounds__(DD_THREADS, 3) delta_decode_kernel(const T* __
   float* lr = gate_s + Dv;               // [rank_a + rank_g]
   float* ws = lr + s.rank_a + s.rank_g;  // [2 * NW]
   float* red = ws + 2 * NW;              // [groups * Dv]
-  float* low = red + groups * Dv;        // [NW][D + Dv]
+  float* low = red;                      // [NW / 2][D + Dv], before red is used
   const int pos = pos_[b], slot = slots[b], hk = h / (s.H / s.Hk);
   const T* row = proj + (size_t)b * ld;
   float* ring = ring0 + (size_t)slot * s.taps * s.channels;
@@ -536,18 +536,20 @@ __global__ void __launch_bounds__(DD_THREADS, 3) delta_decode_kernel(const T* __
   }
   // everything later phases read from global memory is requested here, so that the waits overlap: small vectors, and this
   // thread's first rows of the low-rank matrices
-  constexpr int VW = 16 / sizeof(TW), PRE = 8;
-  const int dg = (D + VW - 1) / VW, vg = (Dv + VW - 1) / VW;
+  // Low-rank products: warps 0..3 work on the decay's second matrix, 4..7 on the gate's (both stored transposed: [rank, heads *
+  // channels]); a lane adds VW neighbouring channels over the rows of its group.
+  constexpr int VW = 16 / sizeof(TW), PRE = 4, LW = NW / 2;
+  const bool is_a = warp < LW;
+  const int lw = is_a ? D : Dv, lrank = is_a ? s.rank_a : s.rank_g, lld = is_a ? a2_ld : g2_ld;
+  const int pieces = (lw + VW - 1) / VW, lpr = pieces <= 16 ? 16 : 32, lrows = LW * (32 / lpr);   // rows per step of the four warps
+  const int lrow0 = (warp % LW) * (32 / lpr) + lane / lpr, lp0 = lane % lpr;
+  const TW* lmat = is_a ? a2t + h * D : g2t + h * Dv;
   const bool vec = D % VW == 0 && Dv % VW == 0;   // rows are 16-byte multiples, so every piece is aligned
-  const bool pre_a = lane < dg;
-  const int pre_c = (pre_a ? lane : lane - dg) * VW, pre_rank = pre_a ? s.rank_a : s.rank_g;
-  const TW* pre_w = (pre_a ? a2t + h * D : g2t + h * Dv) + pre_c;
-  const int pre_ld = pre_a ? a2_ld : g2_ld;
   uint4 pre[PRE];
 #pragma unroll
   for (int i = 0; i < PRE; ++i) {
-    const int r = warp + i * NW;
-    pre[i] = (vec && lane < dg + vg && r < pre_rank) ? *reinterpret_cast<const uint4*>(pre_w + (size_t)r * pre_ld) : make_uint4(0, 0, 0, 0);
+    const int r = lrow0 + i * lrows;
+    pre[i] = (vec && lp0 < pieces && r < lrank) ? *reinterpret_cast<const uint4*>(lmat + (size_t)r * lld + lp0 * VW) : make_uint4(0, 0, 0, 0);
   }
   const float a_log = A_log[h], b_in = dr_ld(row + s.off_b + h), bias0 = tid < D ? dt_bias[h * D + tid] : 0.f, nw0 = tid < Dv ? norm_w[tid] : 0.f;
   if (pos == 0)
@@ -591,47 +593,44 @@ __global__ void __launch_bounds__(DD_THREADS, 3) delta_decode_kernel(const T* __
   float nq2 = 0.f, nk2 = 0.f;
   for (int i = 0; i < NW; ++i) { nq2 += ws[i]; nk2 += ws[NW + i]; }
   const float rq = 1.0f / sqrtf(nq2 + 1e-6f) * (1.0f / sqrtf((float)D)), rk = 1.0f / sqrtf(nk2 + 1e-6f);
-  // low-rank decay and output gate (their second matrices are stored transposed: [rank, heads * channels]): a thread adds VW
-  // neighbouring channels over every eighth rank row, and the eight partial sums meet in shared memory
   const float ea = expf(a_log);
-  for (int p = lane; p < dg + vg; p += 32) {
-    const bool is_a = p < dg;
-    const int c = (is_a ? p : p - dg) * VW, width = is_a ? D : Dv, rank = is_a ? s.rank_a : s.rank_g, ldw = is_a ? a2_ld : g2_ld;
-    const TW* w = (is_a ? a2t + h * D : g2t + h * Dv) + c;
-    const float* f = lr + (is_a ? 0 : s.rank_a);
+  const float* lf = lr + (is_a ? 0 : s.rank_a);
+  for (int p = lp0; p < (pieces + lpr - 1) / lpr * lpr; p += lpr) {   // the same number of turns for every lane
+    const int c = p * VW;
     float a[VW];
 #pragma unroll
     for (int j = 0; j < VW; ++j) a[j] = 0.f;
-    int r0 = warp;
-    if (vec) {
-      if (p == lane) {                             // the rows requested at the start
+    int r0 = lrow0;
+    if (vec && p < pieces) {
+      if (p == lp0) {                              // the rows requested at the start
 #pragma unroll
-        for (int i = 0; i < PRE; ++i) {
-          const float fr = warp + i * NW < rank ? f[warp + i * NW] : 0.f;
-          fma_row(pre[i], fr, a, TW());
-        }
-        r0 += PRE * NW;
+        for (int i = 0; i < PRE; ++i) fma_row(pre[i], lrow0 + i * lrows < lrank ? lf[lrow0 + i * lrows] : 0.f, a, TW());
+        r0 += PRE * lrows;
       }
 #pragma unroll 8
-      for (int r = r0; r < rank; r += NW) {
-        const uint4 raw = *reinterpret_cast<const uint4*>(w + (size_t)r * ldw);
-        fma_row(raw, f[r], a, TW());
+      for (int r = r0; r < lrank; r += lrows) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(lmat + (size_t)r * lld + c);
+        fma_row(raw, lf[r], a, TW());
       }
-    } else {
-      for (int r = r0; r < rank; r += NW)
+    } else if (p < pieces) {
+      for (int r = r0; r < lrank; r += lrows)
 #pragma unroll
         for (int j = 0; j < VW; ++j)
-          if (c + j < width) a[j] = fmaf(dr_ld(w + (size_t)r * ldw + j), f[r], a[j]);
+          if (c + j < lw) a[j] = fmaf(dr_ld(lmat + (size_t)r * lld + c + j), lf[r], a[j]);
     }
+    if (lpr == 16)
 #pragma unroll
-    for (int j = 0; j < VW; ++j)
-      if (c + j < width) low[warp * (D + Dv) + (is_a ? 0 : D) + c + j] = a[j];
+      for (int j = 0; j < VW; ++j) a[j] += __shfl_xor_sync(0xffffffffu, a[j], 16);
+    if (lane < lpr)
+#pragma unroll
+      for (int j = 0; j < VW; ++j)
+        if (c + j < lw) low[(warp % LW) * (D + Dv) + (is_a ? 0 : D) + c + j] = a[j];
   }
   __syncthreads();
   for (int d = tid; d < D + Dv; d += DD_THREADS) {
     float a = 0.f;
 #pragma unroll
-    for (int i = 0; i < NW; ++i) a += low[i * (D + Dv) + d];
+    for (int i = 0; i < LW; ++i) a += low[i * (D + Dv) + d];
     if (d < D) {
       g_s[d] = expf(-ea * dr_softplus(a + (d == tid ? bias0 : dt_bias[h * D + d])));
       q_s[d] *= rq;
@@ -732,8 +731,8 @@ static int launch_delta_decode(const void* proj, int ld, const float* taps_w, fl
                                const float* A_log, const float* dt_bias, const void* a2t, int a2_ld, const void* g2t, int g2_ld,
                                const float* norm_w, float eps, void* out, int out_ld, int B, int* status, const DeltaShape& s, cudaStream_t st) {
   const int lanes_per_row = (s.Dv / VEC + 31) & ~31, groups = DD_THREADS / lanes_per_row;
-  const size_t smem = (size_t)(((s.D * s.Dv + 3) & ~3) + 3 * s.D + 2 * s.Dv + s.rank_a + s.rank_g + 2 * (DD_THREADS / 32) + groups * s.Dv +
-                                (DD_THREADS / 32) * (s.D + s.Dv)) * 4;
+  const size_t smem = (size_t)(((s.D * s.Dv + 3) & ~3) + 3 * s.D + 2 * s.Dv + s.rank_a + s.rank_g + 2 * (DD_THREADS / 32) +
+                                max(groups * s.Dv, DD_THREADS / 64 * (s.D + s.Dv))) * 4;
   if (s.D * s.Dv * 4 > DD_MAX_TILE || smem > 226 * 1024) return -ERR_BAD_ARG;
   static bool configured = false;
   if (!configured) {

@@ -3,8 +3,7 @@
 // Per token the residual is S rows of E floats (fp32, [T, S, E]). A sublayer with output y updates every stream from
 // the old ones, x_t <- sum_s mix[s, t] x_s + out[t] y, and the next sublayer reads LayerNorm(sum_s in[s] x_s). One launch
 // does: (first call of a step) embedding lookup and scaling into the streams, or the update with y; then the weighted
-// sum, the LayerNorm, and the cast to the projections' type. It also clears the split-K accumulators that the previous
-// sublayer's kernels have finished reading. A plain pre-norm residual is S = 1 with unit weights.
+// sum, the LayerNorm, and the cast to the projections' type. A plain pre-norm residual is S = 1 with unit weights.
 //
 // One CTA per token; the row lives in registers (streams) and shared memory (the weighted sum), so the streams are read
 // once and written once: 2 S E 4 bytes per token, the bound of this kernel.
@@ -24,7 +23,6 @@ struct HyperParams {
   float scale;
   const void* y;            // [T, y_ld] sublayer output, or null
   int y_ld;
-  int zero_y;
   const float* mix;         // [S, S], index [from, to]
   const float* out_w;       // [S]
   const float* in_w;        // [S]; null: no normed output is wanted
@@ -35,8 +33,6 @@ struct HyperParams {
   int h_ld;
   const int* rows;          // token of each output row, or null (identity)
   int write_x;
-  float* zero;              // [T, zero_ld] accumulator to clear, or null
-  int zero_ld, zero_n;
   int S, E;
 };
 
@@ -134,10 +130,6 @@ __global__ void __launch_bounds__(NS > 0 ? 512 : 256) hyper_step_kernel(const Hy
         if (t < S)
 #pragma unroll
           for (int j = 0; j < V; ++j) xs[t][j] = nx[t][j];
-      if (p.zero_y) {
-        const float z[4] = {0.f, 0.f, 0.f, 0.f};
-        Vec<YT, V>::st(const_cast<void*>(p.y), row * (size_t)p.y_ld + e, z);
-      }
     }
     if (p.write_x)
 #pragma unroll
@@ -156,10 +148,6 @@ __global__ void __launch_bounds__(NS > 0 ? 512 : 256) hyper_step_kernel(const Hy
       }
       Vec<float, V>::st(hc_u, e, u);
     }
-  }
-  if (p.zero) {
-    float* z = p.zero + row * (size_t)p.zero_ld;
-    for (int i = tid; i < p.zero_n; i += blockDim.x) z[i] = 0.f;
   }
   if (!p.in_w) return;
   const float mean = hc_block_sum(sum, red) / (float)E;
@@ -218,13 +206,12 @@ using namespace inv;
 
 // Types: y_f32 / h_f32 say whether y and h (and the embedding table) are fp32, otherwise bf16 (h fp32 needs y fp32).
 extern "C" int inv_hyper_step(float* x, const int* ids, const void* table, int table_ld, float scale, const void* y, int y_ld, int y_f32,
-                              int zero_y, const float* mix, const float* out_w, const float* in_w, const float* norm_w, const float* norm_b,
-                              float eps, void* h, int h_ld, int h_f32, const int* rows, int n, int write_x, float* zero, int zero_ld,
-                              int zero_n, int S, int E, void* stream) {
+                              const float* mix, const float* out_w, const float* in_w, const float* norm_w, const float* norm_b,
+                              float eps, void* h, int h_ld, int h_f32, const int* rows, int n, int write_x, int S, int E, void* stream) {
   if (S < 1 || S > HC_MAX_STREAMS || E < 1 || E > HC_MAX_WIDTH) return -ERR_BAD_ARG;
   if (h_f32 && !y_f32) return -ERR_BAD_ARG;
   if (n <= 0) return 0;
-  HyperParams p{x, ids, table, table_ld, scale, y, y_ld, zero_y, mix, out_w, in_w, norm_w, norm_b, eps, h, h_ld, rows, write_x, zero, zero_ld, zero_n, S, E};
+  HyperParams p{x, ids, table, table_ld, scale, y, y_ld, mix, out_w, in_w, norm_w, norm_b, eps, h, h_ld, rows, write_x, S, E};
   cudaStream_t st = (cudaStream_t)stream;
   const bool vec = E % 4 == 0 && (!y || y_ld % 4 == 0) && (!in_w || h_ld % 4 == 0) && (!ids || table_ld % 4 == 0);
   if (h_f32) return vec ? hyper_launch<float, float, 4>(p, n, st) : hyper_launch<float, float, 1>(p, n, st);

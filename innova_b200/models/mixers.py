@@ -1,24 +1,23 @@
 """Sequence mixers and feed-forward of the layer-list decoders, as modules with fused, padded weights.
 
 A module is built for one set of sizes, loads its tensors by name (``load``), gives them back under the same names
-(``export``), and runs on packed tokens (``run(ctx, h, cache_index)``). ``ctx`` is the step (``StepContext``): it owns the
-projections' precision and the split-K accumulators of decode steps.
+(``export``), and runs on packed tokens (``run(ctx, h, cache_index)``). ``ctx`` is the step (``StepContext``): it chooses the
+projections' precision and kernel.
 
 Weights of the projections are kept in the model's type with rows padded to 16 bytes; everything that enters a norm, a
 convolution, a decay or a residual is fp32."""
 from __future__ import annotations
 
-from typing import Dict, Optional
+from typing import Dict
 
 import torch
 import torch.nn as nn
 import torch.nn.functional as F
 
-from .. import ops
 from ..ops import delta_rule as dr
 from ..ops import latent_attention as la
-from ..ops.gemm import EPI_ATOMIC, gemm
-from ..ops.hyper import gated_silu, row_buffer
+from ..ops.gemm import SKINNY_ROWS, gemm, skinny_gemm
+from ..ops.hyper import gated_silu
 
 
 def pad_to(n: int, m: int) -> int:
@@ -43,41 +42,28 @@ def put(p: Proj, w: torch.Tensor, row: int = 0):
 
 
 class StepContext:
-    """Precision and scratch of one forward step. In bf16 decode steps the projections are split over K into fp32
-    accumulators that the consuming kernels leave zeroed (``acc``); otherwise they write tensors of their own."""
-
-    ACC_ROWS = 64
+    """Precision of one forward step. bf16 steps of at most 64 rows (decoding) run their projections through the skinny product
+    and hand fp32 results to the consuming kernels; larger ones run the tiled tcgen05 product and write bf16."""
 
     def __init__(self, model, cache, batch):
-        self.batch, self.cache = batch, cache
-        self.dtype = model.dtype
-        self.acc = model.accumulators(cache.device) if (batch.single and batch.T <= self.ACC_ROWS and model.can_accumulate) else None
+        self.batch, self.cache, self.dtype = batch, cache, model.dtype
         self.cuda = cache.device.type == "cuda"
-        self.clear: Optional[torch.Tensor] = None      # accumulator columns the running sublayer has to leave zeroed
+        self.skinny = self.cuda and self.dtype == torch.bfloat16 and batch.single and batch.T <= SKINNY_ROWS
 
     def project(self, x: torch.Tensor, p: Proj, out_dtype=None) -> torch.Tensor:
-        """[T, k] -> [T, padded n] (views of the whole padded rows)."""
+        """[T, k] -> [T, padded n] (whole padded rows)."""
         w = p.weight[:, : p.k]
         if self.cuda and self.dtype == torch.bfloat16:
+            if self.skinny or (x.shape[0] <= SKINNY_ROWS and out_dtype == torch.float32):
+                return skinny_gemm(x[:, : p.k], w)
             return gemm(x[:, : p.k], w, out_dtype=out_dtype or torch.bfloat16)
         return F.linear(x[:, : p.k], w).to(out_dtype or self.dtype)
 
-    def project_in(self, x: torch.Tensor, p: Proj) -> torch.Tensor:
-        """First projection of a sublayer."""
-        if self.acc is None:
-            return self.project(x, p)
-        out = self.acc[0][: x.shape[0], : p.weight.shape[0]]
-        gemm(x[:, : p.k], p.weight[:, : p.k], out=out, epilogue=EPI_ATOMIC)
-        self.clear = out
-        return out
-
-    def project_out(self, x: torch.Tensor, p: Proj) -> torch.Tensor:
-        """Last projection of a sublayer: its result goes into the residual."""
-        if self.acc is None:
-            return self.project(x, p)
-        out = self.acc[1][: x.shape[0], : p.weight.shape[0]]
-        gemm(x[:, : p.k], p.weight[:, : p.k], out=out, epilogue=EPI_ATOMIC)
-        return out
+    def gated(self, x: torch.Tensor, p: Proj, ff: int) -> torch.Tensor:
+        """silu(gate x) * (up x) for a projection that holds the gate rows, then (from the middle) the up rows."""
+        if self.skinny:
+            return skinny_gemm(x[:, : p.k], p.weight[:, : p.k], n=ff, silu_half=p.n // 2, out_dtype=torch.bfloat16)
+        return gated_silu(self.project(x, p), ff, self.dtype)
 
 
 class LatentAttention(nn.Module):
@@ -108,9 +94,6 @@ class LatentAttention(nn.Module):
     def latent(self):
         return self.Rp, self.window
 
-    def in_width(self) -> int:
-        return self.inp.weight.shape[0]
-
     @torch.no_grad()
     def load(self, t: Dict[str, torch.Tensor], p: str):
         H, D, Dv, Dp, R = self.H, self.D, self.Dv, self.Dp, self.R
@@ -140,7 +123,7 @@ class LatentAttention(nn.Module):
     def run(self, ctx: StepContext, h: torch.Tensor, index: int) -> torch.Tensor:
         b, cache = ctx.batch, ctx.cache
         pool, T, nq = cache.latent[index], h.shape[0], self.off_c
-        qc = ctx.project_in(h, self.inp)
+        qc = ctx.project(h, self.inp)
         flash = ctx.cuda and ctx.dtype == torch.bfloat16 and b.fresh and not b.single and self.Dp <= 128
         c, q = la.latent_append(qc, nq, self.R, self.norm, self.eps, pool, cache.page_table, b, want_c=flash,
                                 nq=nq if qc.dtype != pool.dtype else 0)
@@ -152,7 +135,7 @@ class LatentAttention(nn.Module):
             span = min(self.window or cache.max_pages * la.PAGE, cache.max_pages * la.PAGE)
             lat = la.latent_attend(la.head_proj(q, self.uk), pool, cache.page_table, self.H, self.scale, self.window, b, span)
             o = la.head_proj(lat, self.kv.weight[nq:2 * nq].view(self.H, self.Dp, self.Rp))
-        return ctx.project_out(o, self.out)
+        return ctx.project(o, self.out)
 
 
 class ChannelDelta(nn.Module):
@@ -172,9 +155,6 @@ class ChannelDelta(nn.Module):
         self.A_log, self.dt_bias = frozen(s.H, dtype=torch.float32), frozen(s.H * s.D, dtype=torch.float32)
         self.norm = frozen(s.Dv, dtype=torch.float32)
         self.out = Proj(width, s.H * s.Dv, dtype)
-
-    def in_width(self) -> int:
-        return self.inp.weight.shape[0]
 
     @torch.no_grad()
     def load(self, t: Dict[str, torch.Tensor], p: str):
@@ -214,15 +194,16 @@ class ChannelDelta(nn.Module):
 
     def run(self, ctx: StepContext, h: torch.Tensor, index: int) -> torch.Tensor:
         s, b, cache = self.shape, ctx.batch, ctx.cache
-        proj = ctx.project_in(h, self.inp)
+        proj = ctx.project(h, self.inp)
         args = (self.taps, self.A_log, self.dt_bias, self.norm, self.eps, cache.ring[index], cache.state[index], b)
         if b.single and s.tile_bytes <= dr.DECODE_MAX_TILE:
             o = dr.delta_decode(s, proj, self.a2t, self.g2t, *args)
         else:
-            z = ctx.project(proj[:, s.offsets[3]:], self.a2, torch.float32)
-            gate = ctx.project(proj[:, s.offsets[4]:], self.g2)
+            wide = proj.to(ctx.dtype)      # (a decode step with a state tile too large for the one-launch kernel has fp32 rows)
+            z = ctx.project(wide[:, s.offsets[3]:], self.a2, torch.float32)
+            gate = ctx.project(wide[:, s.offsets[4]:], self.g2).to(ctx.dtype)
             o = dr.delta_prompt(s, proj, z, gate, *args)
-        return ctx.project_out(o, self.out)
+        return ctx.project(o, self.out)
 
 
 class GatedMLP(nn.Module):
@@ -233,9 +214,6 @@ class GatedMLP(nn.Module):
         self.width, self.ff, self.half = width, ff, pad_to(ff, 8)
         self.inp = Proj(2 * self.half, width, dtype)
         self.out = Proj(width, ff, dtype)
-
-    def in_width(self) -> int:
-        return self.inp.weight.shape[0]
 
     @torch.no_grad()
     def load(self, t, p):
@@ -248,7 +226,7 @@ class GatedMLP(nn.Module):
                 p + "down": self.out.weight[: self.width, : self.ff]}
 
     def run(self, ctx: StepContext, h: torch.Tensor, index: int = 0) -> torch.Tensor:
-        return ctx.project_out(gated_silu(ctx.project_in(h, self.inp), self.ff, ctx.dtype), self.out)
+        return ctx.project(ctx.gated(h, self.inp, self.ff), self.out)
 
 
 MIXERS = {c.kind: c for c in (LatentAttention, ChannelDelta)}

@@ -16,7 +16,6 @@ import torch
 import torch.nn as nn
 
 from ..inference.state_cache import LatentStateCache, StepBatch
-from ..ops import delta_rule as dr
 from ..ops.gemm import full_fp32_matmul
 from ..ops.hyper import HyperIn, HyperOut, hyper_step
 from .mixers import MIXERS, GatedMLP, Proj, StepContext, frozen, put
@@ -104,7 +103,7 @@ class Sublayer(nn.Module):
 @register("Vebesun")
 class VebesunModel(nn.Module):
     # what a fresh checkout compiles to run this model
-    CUDA_SOURCES = ("hyper.cu", "delta_rule.cu", "latent_attn.cu", "flash_attn_fwd.cu", "gemm_tcgen05.cu", "gemm_tcgen05_2cta.cu", "elementwise.cu",
+    CUDA_SOURCES = ("hyper.cu", "delta_rule.cu", "latent_attn.cu", "skinny_gemm.cu", "flash_attn_fwd.cu", "gemm_tcgen05.cu", "gemm_tcgen05_2cta.cu", "elementwise.cu",
                     "sampler.cu")
     HOST_SOURCES = ("importers.cpp",)
     config_class = VebesunConfig
@@ -132,9 +131,6 @@ class VebesunModel(nn.Module):
             kind = cfg.layers[i]["type"]
             self.runs.append((i, counts.setdefault(kind, 0)))
             counts[kind] += 1
-        self.can_accumulate = dtype == torch.bfloat16 and all(
-            m.body.shape.tile_bytes <= dr.DECODE_MAX_TILE for m in self.modules() if isinstance(m, Sublayer) and hasattr(m.body, "shape"))
-        self._acc = None
         if seed is not None:
             self.reset_parameters(seed)
         if device is not None:
@@ -228,16 +224,6 @@ class VebesunModel(nn.Module):
                 states.append(body.shape)
         return LatentStateCache(latents, states, max_batch, max_seq, device or self.embed.weight.device, self.dtype, num_pages)
 
-    def accumulators(self, device):
-        """Two fp32 split-K accumulators (first and last projection of a sublayer), zero between kernels."""
-        if device.type != "cuda":
-            return None
-        if self._acc is None:
-            wide = max(s.body.in_width() for l in self.layers for s in l)
-            rows, E = StepContext.ACC_ROWS, self.embed.weight.shape[1]
-            self._acc = (torch.zeros(rows, wide, dtype=torch.float32, device=device), torch.zeros(rows, E, dtype=torch.float32, device=device))
-        return self._acc
-
     @torch.no_grad()
     def step(self, cache: LatentStateCache, batch: StepBatch, hidden: bool = False, residuals: Optional[list] = None):
         """Run the batch's new tokens; returns fp32 logits [wanted, vocab] (or the final normed states with ``hidden``), None when
@@ -257,9 +243,7 @@ class VebesunModel(nn.Module):
                 h = hyper_step(x, self.dtype, prev, nxt, batch.ids if first else None, table if first else None, cfg.embedding_scale)
                 if residuals is not None and q == 0 and run > 0:
                     residuals.append(x.sum(1))
-                ctx.clear = None
-                y = sub.body.run(ctx, h, index)
-                prev = HyperOut(y, sub.mix, sub.outw, clear_y=ctx.acc is not None, clear=ctx.clear)
+                prev = HyperOut(sub.body.run(ctx, h, index), sub.mix, sub.outw)
         if prev is None:               # no layers at all
             hyper_step(x, self.dtype, None, None, batch.ids, table, cfg.embedding_scale)
         head = HyperIn(self.ones, self.final_w, self.final_b, cfg.norm_eps)

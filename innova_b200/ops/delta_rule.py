@@ -105,7 +105,7 @@ def delta_prompt(s: DeltaShape, proj, z, gate, taps_w, A_log, dt_bias, norm_w, e
 
 
 def delta_decode(s: DeltaShape, proj, a2t, g2t, taps_w, A_log, dt_bias, norm_w, eps, ring, state, batch) -> torch.Tensor:
-    """One token per sequence in one launch: ``proj`` [B, width] (type of the weights, or fp32 accumulators) -> [B, H * Dv] in the
+    """One token per sequence in one launch: ``proj`` [B, width] (type of the weights, or fp32) -> [B, H * Dv] in the
     type of ``a2t`` [rank_a, H * D] / ``g2t`` [rank_g, H * Dv], the transposed second factors of the low-rank products."""
     B = proj.shape[0]
     if not proj.is_cuda:

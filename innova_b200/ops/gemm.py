@@ -15,6 +15,7 @@ import contextlib
 import torch
 import torch.nn.functional as F
 
+from .. import _native
 from . import runtime as rt
 
 EPI_NONE, EPI_GELU, EPI_DGELU, EPI_ADD, EPI_ATOMIC, EPI_GELU_DG, EPI_MUL = 0, 1, 2, 3, 4, 5, 6
@@ -97,6 +98,22 @@ def gemm(a, b, out=None, *, a_mn=False, b_mn=False, M=None, N=None, K=None, epil
         rt.status_tensor(a.device).data_ptr(), rt.stream_ptr(), _kernel_select)
     rt.check(rc, "inv_gemm_bf16")
     return out
+
+
+_native.register_cuda_sigs({"inv_skinny_gemm": [_native.vp, _native.i32, _native.vp] + [_native.i32] * 5 + [_native.vp, _native.i32, _native.i32, _native.vp]})
+SKINNY_ROWS = 64
+
+
+def skinny_gemm(x, w, n=None, silu_half: int = 0, out_dtype=torch.float32):
+    """x [M <= 64, K] times w [N, K]^T for decode steps (csrc/skinny_gemm.cu): weights straight from memory into MMA fragments,
+    no tile set-up. Rows of both operands start on 16-byte boundaries. ``silu_half``: w holds gate rows [0, n) and up rows
+    [silu_half, silu_half + n) and the result is silu(gate) * up."""
+    M, K = x.shape
+    n = w.shape[0] if n is None else n
+    out = torch.empty((M, (n + 7) // 8 * 8), dtype=out_dtype, device=x.device)
+    rt.check(rt.lib().inv_skinny_gemm(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), M, n, K, silu_half, out.data_ptr(), out.stride(0),
+                                      int(out_dtype == torch.float32), rt.stream_ptr()), "inv_skinny_gemm")
+    return out[:, :n]
 
 
 def _accumulate_wgrad(weight, dy2, x2):

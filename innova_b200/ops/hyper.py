@@ -17,7 +17,7 @@ from . import runtime as rt
 
 _vp, _i, _f = _native.vp, _native.i32, _native.f32
 _native.register_cuda_sigs({
-    "inv_hyper_step": [_vp, _vp, _vp, _i, _f, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _f, _vp, _i, _i, _vp, _i, _i, _vp, _i, _i, _i, _i, _vp],
+    "inv_hyper_step": [_vp, _vp, _vp, _i, _f, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _f, _vp, _i, _i, _vp, _i, _i, _i, _i, _vp],
     "inv_gated_silu_f32": [_vp, _i, _i, _vp, _i, _i, _i, _i, _vp],
 })
 
@@ -28,8 +28,6 @@ class HyperOut:
     y: torch.Tensor                          # [T, >= E] fp32 or bf16
     mix: torch.Tensor                        # [S, S] fp32, index [from, to]
     out: torch.Tensor                        # [S] fp32
-    clear_y: bool = False                    # y is an accumulator: leave zeros behind
-    clear: Optional[torch.Tensor] = None     # [T, n] view of another accumulator to leave zeroed
 
 
 @dataclass
@@ -56,15 +54,14 @@ def hyper_step(x: torch.Tensor, dtype, prev: Optional[HyperOut] = None, nxt: Opt
         return _hyper_step_cpu(x, dtype, prev, nxt, ids, table, scale, rows, keep)
     n = T if rows is None else rows.numel()
     h = row_buffer(n, E, dtype, x.device) if nxt is not None else None
-    y, clear = (prev.y, prev.clear) if prev is not None else (None, None)
+    y = prev.y if prev is not None else None
     table_ld = table.stride(0) if ids is not None else 0
     rc = rt.lib().inv_hyper_step(
         x.data_ptr(), rt.ptr(ids), rt.ptr(table) if ids is not None else 0, table_ld, float(scale), rt.ptr(y), 0 if y is None else y.stride(0),
-        int(dtype == torch.float32 if y is None else y.dtype == torch.float32), int(prev is not None and prev.clear_y and rows is None),
+        int(dtype == torch.float32 if y is None else y.dtype == torch.float32),
         rt.ptr(prev.mix) if prev else 0, rt.ptr(prev.out) if prev else 0, rt.ptr(nxt.weight) if nxt else 0, rt.ptr(nxt.norm_w) if nxt else 0,
         rt.ptr(nxt.norm_b) if nxt else 0, float(nxt.eps) if nxt else 0.0, rt.ptr(h), 0 if h is None else h.stride(0), int(dtype == torch.float32),
-        rt.ptr(rows), n, int(keep), rt.ptr(clear) if rows is None else 0, 0 if clear is None else clear.stride(0),
-        0 if clear is None else clear.shape[1], S, E, rt.stream_ptr())
+        rt.ptr(rows), n, int(keep), S, E, rt.stream_ptr())
     rt.check(rc, "inv_hyper_step")
     return h
 
@@ -88,7 +85,7 @@ def _hyper_step_cpu(x, dtype, prev, nxt, ids, table, scale, rows, keep):
 
 def gated_silu(gate_up: torch.Tensor, n: int, dtype) -> torch.Tensor:
     """silu(gate) * up from rows that hold n gate columns (padded to the row's half), then n up columns. bf16 rows take the
-    training activation kernel; fp32 rows (32-bit models and split-K accumulators) the one in ``csrc/hyper.cu``."""
+    training activation kernel; fp32 rows (32-bit models) the one in ``csrc/hyper.cu``."""
     T, half = gate_up.shape[0], gate_up.shape[1] // 2
     if not gate_up.is_cuda:
         return (F.silu(gate_up[:, :n].float()) * gate_up[:, half:half + n].float()).to(dtype)

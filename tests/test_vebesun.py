@@ -129,14 +129,16 @@ def test_hyper_step(dev, S, E):
 
 
 @pytest.mark.gpu
-def test_hyper_step_clears_accumulators():
-    x = torch.randn(5, 2, 40, device="cuda")
-    acc_in, acc_y = torch.randn(8, 96, device="cuda"), torch.randn(8, 40, device="cuda")
-    keep = acc_in.clone()
-    one = torch.ones(2, device="cuda")
-    hyper_step(x, torch.bfloat16, HyperOut(acc_y[:5], torch.eye(2, device="cuda"), one, True, acc_in[:5, :64]))
-    assert not acc_y[:5].any() and acc_y[5:].any() and not acc_in[:5, :64].any()
-    assert torch.equal(acc_in[:, 64:], keep[:, 64:]) and torch.equal(acc_in[5:], keep[5:])
+@pytest.mark.parametrize("M", [1, 7, 16, 17, 40, 64])
+@pytest.mark.parametrize("N,K", [(48, 96), (53, 52), (256, 1000), (5000, 128), (8, 20)])
+def test_skinny_product(M, N, K):
+    from innova_b200.ops import skinny_gemm
+    pad = lambda a: torch.nn.functional.pad(a, (0, -a.shape[1] % 8), value=float("nan")).cuda().bfloat16()      # padding is never used
+    x, w = pad(torch.randn(M, K))[:, :K], pad(torch.randn(2 * N, K) * K ** -0.5)[:, :K]
+    want = x.double() @ w.double().t()
+    assert torch.allclose(skinny_gemm(x, w[:N]).double(), want[:, :N], atol=2e-4, rtol=1e-3)
+    got = skinny_gemm(x, w, n=N - 3, silu_half=N, out_dtype=torch.bfloat16).double()
+    assert torch.allclose(got, oracle.silu(want[:, :N - 3]) * want[:, N:2 * N - 3], atol=3e-2, rtol=2e-2)
 
 
 @pytest.mark.parametrize("F", [24, 19])
@@ -247,7 +249,7 @@ def test_delta_rule_prompts_portions_and_decoding(dev, s):
 
 
 @pytest.mark.gpu
-def test_delta_decode_reads_fp32_accumulators():
+def test_delta_decode_reads_fp32_rows():
     s = SHAPES[2]
     p = delta_params(s, torch.bfloat16)
     x = delta_inputs(s, 3, 1, torch.float32)
