@@ -16,7 +16,7 @@ import torch.nn.functional as F
 
 from ..ops import delta_rule as dr
 from ..ops import latent_attention as la
-from ..ops.gemm import SKINNY_ROWS, gemm, skinny_gemm
+from ..ops.gemm import EPI_ATOMIC, NUM_SMS, SKINNY_ROWS, gemm, skinny_gemm
 from ..ops.hyper import gated_silu
 
 
@@ -42,22 +42,30 @@ def put(p: Proj, w: torch.Tensor, row: int = 0):
 
 
 class StepContext:
-    """Precision of one forward step. bf16 steps of at most 64 rows (decoding) run their projections through the skinny product
-    and hand fp32 results to the consuming kernels; larger ones run the tiled tcgen05 product and write bf16."""
+    """Precision of one forward step. bf16 steps of one token per sequence, at most 64 of them, hand fp32 projections to the
+    consuming kernels: up to 32 rows from the skinny product, more from the tiled tcgen05 product split over K. Larger steps run
+    the tiled product and write bf16."""
+
+    SPLIT_ROWS = 64
 
     def __init__(self, model, cache, batch):
         self.batch, self.cache, self.dtype = batch, cache, model.dtype
-        self.cuda = cache.device.type == "cuda"
-        self.skinny = self.cuda and self.dtype == torch.bfloat16 and batch.single and batch.T <= SKINNY_ROWS
+        self.bf16 = cache.device.type == "cuda" and self.dtype == torch.bfloat16
+        self.small = self.bf16 and batch.single and batch.T <= self.SPLIT_ROWS
+        self.skinny = self.small and batch.T <= SKINNY_ROWS
 
     def project(self, x: torch.Tensor, p: Proj, out_dtype=None) -> torch.Tensor:
         """[T, k] -> [T, padded n] (whole padded rows)."""
-        w = p.weight[:, : p.k]
-        if self.cuda and self.dtype == torch.bfloat16:
-            if self.skinny or (x.shape[0] <= SKINNY_ROWS and out_dtype == torch.float32):
-                return skinny_gemm(x[:, : p.k], w)
-            return gemm(x[:, : p.k], w, out_dtype=out_dtype or torch.bfloat16)
-        return F.linear(x[:, : p.k], w).to(out_dtype or self.dtype)
+        x, w = x[:, : p.k], p.weight[:, : p.k]
+        if not self.bf16:
+            return F.linear(x, w).to(out_dtype or self.dtype)
+        rows, n = x.shape[0], w.shape[0]
+        if self.skinny or (rows <= SKINNY_ROWS and out_dtype == torch.float32):
+            return skinny_gemm(x, w)
+        if self.small and (n + 255) // 256 <= NUM_SMS // 2:
+            out = torch.zeros(rows, n, dtype=torch.float32, device=x.device)
+            return gemm(x, w, out=out, epilogue=EPI_ATOMIC, split_k=max(1, NUM_SMS // ((n + 255) // 256)))
+        return gemm(x, w, out_dtype=torch.float32 if self.small else (out_dtype or torch.bfloat16))
 
     def gated(self, x: torch.Tensor, p: Proj, ff: int) -> torch.Tensor:
         """silu(gate x) * (up x) for a projection that holds the gate rows, then (from the middle) the up rows."""
@@ -124,7 +132,7 @@ class LatentAttention(nn.Module):
         b, cache = ctx.batch, ctx.cache
         pool, T, nq = cache.latent[index], h.shape[0], self.off_c
         qc = ctx.project(h, self.inp)
-        flash = ctx.cuda and ctx.dtype == torch.bfloat16 and b.fresh and not b.single and self.Dp <= 128
+        flash = ctx.bf16 and b.fresh and not b.single and self.Dp <= 128
         c, q = la.latent_append(qc, nq, self.R, self.norm, self.eps, pool, cache.page_table, b, want_c=flash,
                                 nq=nq if qc.dtype != pool.dtype else 0)
         q = qc[:, :nq] if q is None else q

@@ -58,6 +58,8 @@ CONFIGS = {
     "loop": config([ff(delta(2, 2, 64, 72, 4), None), ff(attn(2, 16, 96, 64, 1), 64), ff(attn(4, 64, 64, 48, 33), 40)], width=64, streams=4,
                    loop={"start": 0, "stop": 3, "times": 2}, eps=1e-3),
     # heads too large for the flash kernel, a state tile of the largest decode size, five streams
+    # a state tile too large for the one-launch decode kernel, more streams than the unrolled residual kernels, no feed-forward
+    "tile": config([ff(delta(1, 1, 256, 224, 2), None), ff(attn(3, 32, 32, 48, 12), None)], width=48, streams=7),
     "large": config([ff(attn(2, 144, 80, 160, 50), 64), ff(delta(2, 1, 160, 128, 4), 48)], width=128, streams=5),
 }
 
@@ -377,6 +379,28 @@ def test_unequal_requests_and_reused_rows(dev):
         for r in rows:
             gen.cache.free(r)
         assert len(gen.cache._free) == gen.cache.num_pages
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("n", [20, 40, 70])
+@pytest.mark.parametrize("name", ["mixed", "large", "tile"])
+def test_wide_decode_batches(name, n):
+    """Projections change kernels with the number of rows: up to 32, up to 64, more."""
+    cfg = CONFIGS[name]
+    for dt in (torch.float32, torch.bfloat16):
+        model, w = build(cfg, ("cuda", dt), 14)
+        seqs = [tokens(3 + i % 5, cfg, i % 7) + tokens(3, cfg, 90 + i % 3) for i in range(n)]
+        known = {}
+        gen = Generator(model, max_batch=n, max_seq=32)
+        gen.use_graphs = False
+        at = [len(s) - 3 for s in seqs]
+        gen.step([s[:p] for s, p in zip(seqs, at)], [0] * n, list(range(n)))
+        for k in range(3):
+            lg = gen.step([[s[p + k]] for s, p in zip(seqs, at)], [p + k for p in at], list(range(n)))
+            for i, s in enumerate(seqs):
+                if tuple(s) not in known:
+                    known[tuple(s)] = oracle.forward(cfg, w, s)
+            assert error(lg, torch.stack([known[tuple(s)][p + k] for s, p in zip(seqs, at)])) < tol(("cuda", dt))
 
 
 def test_pages_behind_every_window_are_given_back():
