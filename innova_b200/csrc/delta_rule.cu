@@ -844,7 +844,7 @@ extern "C" int inv_gated_head_norm(const float* o, const float* w, const void* g
 }
 
 // One token per sequence. Weights a2t [rank_a, a2_ld], g2t [rank_g, g2_ld] and out are bf16 (act_f32 = 0) or fp32; proj may be
-// fp32 with bf16 weights (split-K accumulators). A state tile larger than DD_MAX_TILE is refused (use the prompt path).
+// fp32 with bf16 weights. A state tile larger than DD_MAX_TILE is refused (use the prompt path).
 extern "C" int inv_delta_decode(const void* proj, int ld, int proj_f32, const float* taps_w, float* ring, float* state, const int* pos,
                                 const int* slots, const float* A_log, const float* dt_bias, const void* a2t, int a2_ld, const void* g2t, int g2_ld,
                                 int act_f32, const float* norm_w, float eps, void* out, int out_ld, int B, int* status, const int* shape,

@@ -168,7 +168,7 @@ class Rows:
 
 
 SHAPES = [dr.DeltaShape(4, 2, 16, 24, 3, 6, 9), dr.DeltaShape(3, 3, 40, 33, 1, 8, 8), dr.DeltaShape(6, 1, 64, 64, 4, 24, 24), dr.DeltaShape(2, 2, 128, 128, 5, 16, 40),
-          dr.DeltaShape(2, 2, 50, 256, 2, 4, 4), dr.DeltaShape(1, 1, 200, 20, 4, 8, 8)]
+          dr.DeltaShape(2, 2, 50, 256, 2, 4, 4), dr.DeltaShape(1, 1, 200, 20, 4, 8, 8), dr.DeltaShape(4, 2, 32, 16, 9, 7, 130)]
 
 
 def delta_inputs(s, n, seed, dt):
