@@ -146,7 +146,7 @@ def kernel_section(size="2k"):
     """Every kernel of the design alone, and the like kernel of the closest model: time, bytes or FLOPs, fraction of the roofline."""
     from innova_b200 import ops
     from innova_b200.inference.kv_cache import PagedKVCache
-    from innova_b200.inference.state_cache import LatentStateCache, StepBatch
+    from innova_b200.inference.state_cache import Latents, StepBatch, StepCache
     from innova_b200.ops import delta_rule as dr
     from innova_b200.ops import latent_attention as la
     from innova_b200.ops import runtime as rt
@@ -191,7 +191,7 @@ def kernel_section(size="2k"):
     lens = {"1x8192": [8192], "16x1024": [1024] * 16}
     for name, ls in lens.items():
         T = sum(ls)
-        c = LatentStateCache([], [s], len(ls), max(ls) + 16, dev)
+        c = StepCache(len(ls), max(ls) + 16, dev, states=[s])
         for i, n in enumerate(ls):
             c.reserve(i, n)
         b = StepBatch(c, [[0] * n for n in ls], [0] * len(ls), list(range(len(ls))))
@@ -218,7 +218,7 @@ def kernel_section(size="2k"):
         report("gated_head_norm", f"{name} H{H}", cold(hnorm), T * H * 128 * 8 / 1e9)
         del blocks, vblocks, o, proj, z, gate
     for B in (1, 16, 64):
-        c = LatentStateCache([], [s], B, 64, dev)
+        c = StepCache(B, 64, dev, states=[s])
         for i in range(B):
             c.reserve(i, 11)
         b = StepBatch(c, [[0]] * B, [10] * B, list(range(B)))
@@ -228,8 +228,7 @@ def kernel_section(size="2k"):
                (B * H * 128 * 128 * 8 + 2 * RANK * H * 128 * 2 + B * s.offsets[6] * 4 + 3 * B * s.channels * 4) / 1e9)
     # attention, decode: latents against the dense decoder's paged KV cache (bf16) at the same heads and span
     for B in (1, 16, 64):
-        c = LatentStateCache([(R, WINDOW)], [], B, 2048, dev)
-        c.reach = None
+        c = StepCache(B, 2048, dev, latents=[Latents(R, WINDOW)])
         for i in range(B):
             c.reserve(i, 1537)
         b = StepBatch(c, [[0]] * B, [1536] * B, list(range(B)))
@@ -252,7 +251,7 @@ def kernel_section(size="2k"):
         report("gemm", f"M{B} N4096 K{E}", cold(lambda: ops.gemm(xl, wl)), wl.numel() * 2 / 1e9, like="skinny_gemm")
     # attention, prompts
     T = 8192
-    c = LatentStateCache([(R, WINDOW)], [], 1, T, dev)
+    c = StepCache(1, T, dev, latents=[Latents(R, WINDOW)])
     c.reserve(0, T)
     b = StepBatch(c, [[0] * T], [0], [0])
     qkv = rand(1, T, 3 * H * 128).to(bf)

@@ -26,7 +26,7 @@ NVCC_FLAGS = [
     "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-O3",
 ]
 # Sources whose arithmetic also serves the fp32 models: IEEE division and square root, accurate exponentials.
-PRECISE_SOURCES = {"hyper.cu", "delta_rule.cu", "latent_attn.cu", "skinny_gemm.cu"}
+PRECISE_SOURCES = {"hyper.cu", "delta_rule.cu", "latent_attn.cu", "skinny_gemm.cu", "kv_attn.cu", "sandwich.cu"}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function", "-pthread"]
 
 

@@ -32,6 +32,9 @@ struct FlashFwdParams {
   float scale;
   int causal;
   int window;  // > 0 (causal only): a query sees the `window` most recent keys, its own position included
+  int chunk;   // > 0 (causal only): a query sees the earlier keys of its own chunk of `chunk` positions (counted from position 0)
+  const __nv_bfloat16* gate;  // the output is multiplied by sigmoid(gate), element by element; null: no gate
+  int ld_gate;
   const int* cu;  // packed batch: sequence b is rows [cu[b], cu[b + 1]) of the token-major buffers; null: B sequences of S rows
   int* status;
 };
@@ -93,8 +96,9 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
   const int hk = h / (p.H / p.Hkv);
   const int q0 = q_blk * FA_BM;
   const int nkb_all = (S + FA_BN - 1) / FA_BN;
-  // key blocks visited: [jlo, jlo + nkb). A sliding window skips the blocks that lie wholly before the first query's window.
-  const int jlo = (p.causal && p.window > 0) ? max(0, q0 - p.window + 1) / FA_BN : 0;
+  // key blocks visited: [jlo, jlo + nkb). A sliding window skips the blocks that lie wholly before the first query's window, a
+  // chunked mask those before the first query's chunk.
+  const int jlo = !p.causal ? 0 : p.window > 0 ? max(0, q0 - p.window + 1) / FA_BN : p.chunk > 0 ? (q0 - q0 % p.chunk) / FA_BN : 0;
   const int nkb = (p.causal ? min(nkb_all, q_blk + 1) : nkb_all) - jlo;
   constexpr uint32_t TMEM_COLS = ND == 1 ? 256 : 512;
   constexpr uint32_t O_COL = 128, P_COL = 128 + D;
@@ -187,15 +191,17 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     const uint32_t t_lane = tmem_base + (uint32_t(q * 32) << 16);
     const float c = p.scale * 1.4426950408889634f;
     float m_used = -INFINITY, l = 0.f;
+    const bool windowed = p.causal && p.window > 0, chunked = p.causal && p.chunk > 0;
+    const int kmin = windowed ? row - p.window + 1 : chunked ? row - row % p.chunk : 0;
+    const int last = min(q0 + FA_BM, S) - 1;                    // the block's last row has the highest first visible key
+    const int kmin_last = windowed ? last - p.window + 1 : chunked ? last - last % p.chunk : 0;
     bool ok = true;
     for (int j = 0; j < nkb; ++j) {
       if (!mbar_wait_warp(s_full, j & 1, abort_flag, p.status, ERR_WAIT_TMEM_FULL)) { ok = false; break; }
       tc_fence_after();
       const int k0 = (jlo + j) * FA_BN;
-      const bool windowed = p.causal && p.window > 0;
-      const bool need_mask = (p.causal && k0 + FA_BN - 1 > q0) || (k0 + FA_BN > S) || (windowed && k0 <= q0 + FA_BM - 1 - p.window);
+      const bool need_mask = (p.causal && k0 + FA_BN - 1 > q0) || (k0 + FA_BN > S) || k0 < kmin_last;
       const int kmax = p.causal ? min(row, S - 1) : S - 1;
-      const int kmin = windowed ? row - p.window + 1 : 0;
       uint32_t sr[128];
       tmem_ld_32x32(t_lane, sr);
       tmem_ld_32x32(t_lane + 32, sr + 32);
@@ -264,13 +270,28 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     if (ok) {
       tc_fence_after();
       const float inv_l = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* dst = p.out + ((p.cu ? (size_t)row_base : (size_t)b * S) + row) * p.ld_o + h * D;
+      const size_t grow = (p.cu ? (size_t)row_base : (size_t)b * S) + row;
+      __nv_bfloat16* dst = p.out + grow * p.ld_o + h * D;
+      const __nv_bfloat16* gate = p.gate ? p.gate + grow * p.ld_gate + h * D : nullptr;
 #pragma unroll 1
       for (int cc = 0; cc < D / 32; ++cc) {
         uint32_t rr[32];
         tmem_ld_32x32(t_lane + O_COL + cc * 32, rr);
         tmem_ld_wait();
         if (row < S) {
+          if (gate) {
+#pragma unroll
+            for (int g = 0; g < 4; ++g) {
+              const uint4 gv = *reinterpret_cast<const uint4*>(gate + cc * 32 + g * 8);
+              const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+              for (int i = 0; i < 4; ++i) {
+                const float g0 = __uint_as_float(gw[i] << 16), g1 = __uint_as_float(gw[i] & 0xffff0000u);
+                rr[g * 8 + 2 * i] = __float_as_uint(__uint_as_float(rr[g * 8 + 2 * i]) / (1.0f + __expf(-g0)));
+                rr[g * 8 + 2 * i + 1] = __float_as_uint(__uint_as_float(rr[g * 8 + 2 * i + 1]) / (1.0f + __expf(-g1)));
+              }
+            }
+          }
 #pragma unroll
           for (int g = 0; g < 4; ++g) {
             uint4 o;
@@ -347,9 +368,9 @@ using namespace inv;
 
 static int flash_fwd_launch(const void* q, const void* k, const void* v, void* out, float* lse, const int* cu, int n_seq, int max_len, int map_b,
                             int map_s, int H, int Hkv, int head_dim, int ld_q, int ld_k, int ld_v, int ld_o, float scale, int causal, int window,
-                            int* status, void* stream) {
-  if ((head_dim != 64 && head_dim != 128) || H % Hkv || (ld_q % 8) || (ld_k % 8) || (ld_v % 8) || (ld_o % 8)) return -ERR_BAD_ARG;
-  if (window < 0 || (window > 0 && !causal)) return -ERR_BAD_ARG;  // the sliding window is defined for causal attention
+                            int chunk, const void* gate, int ld_gate, int* status, void* stream) {
+  if ((head_dim != 64 && head_dim != 128) || H % Hkv || (ld_q % 8) || (ld_k % 8) || (ld_v % 8) || (ld_o % 8) || (gate && ld_gate % 8)) return -ERR_BAD_ARG;
+  if (window < 0 || chunk < 0 || ((window > 0 || chunk > 0) && !causal) || (window > 0 && chunk > 0)) return -ERR_BAD_ARG;
   if (n_seq <= 0 || max_len <= 0) return 0;
   CUtensorMap tq, tk, tv;
   int rc;
@@ -360,6 +381,8 @@ static int flash_fwd_launch(const void* q, const void* k, const void* v, void* o
   p.out = (__nv_bfloat16*)out; p.ld_o = ld_o; p.lse = lse;
   p.B = n_seq; p.S = max_len; p.H = H; p.Hkv = Hkv; p.scale = scale; p.causal = causal ? 1 : 0; p.status = status; p.cu = cu;
   p.window = window >= max_len ? 0 : window;
+  p.chunk = chunk >= max_len ? 0 : chunk;
+  p.gate = (const __nv_bfloat16*)gate; p.ld_gate = ld_gate;
   dim3 grid((max_len + FA_BM - 1) / FA_BM, H, n_seq);
   cudaStream_t st = (cudaStream_t)stream;
   static bool configured = false;
@@ -379,14 +402,17 @@ static int flash_fwd_launch(const void* q, const void* k, const void* v, void* o
 extern "C" int inv_flash_attn_fwd(const void* q, const void* k, const void* v, void* out, float* lse, int B, int S, int H, int Hkv,
                                   int head_dim, int ld_q, int ld_k, int ld_v, int ld_o, float scale, int causal, int window, int* status,
                                   void* stream) {
-  return flash_fwd_launch(q, k, v, out, lse, nullptr, B, S, B, S, H, Hkv, head_dim, ld_q, ld_k, ld_v, ld_o, scale, causal, window, status, stream);
+  return flash_fwd_launch(q, k, v, out, lse, nullptr, B, S, B, S, H, Hkv, head_dim, ld_q, ld_k, ld_v, ld_o, scale, causal, window, 0, nullptr, 0,
+                          status, stream);
 }
 
 // Packed sequences: rows [cu[i], cu[i + 1]) of [T, ld*] are sequence i (cu: n_seq + 1 device ints, cu[n_seq] = T, none longer
-// than max_len). Causal. A tile that reaches past its sequence reads the next one's rows, which the mask removes.
+// than max_len). Causal, with a window or a chunked mask (not both). A tile that reaches past its sequence reads the next one's
+// rows, which the mask removes. gate: bf16 [T, ld_gate] of the output's columns, or null.
 extern "C" int inv_flash_attn_packed(const void* q, const void* k, const void* v, void* out, const int* cu, int n_seq, int T, int max_len, int H,
-                                     int Hkv, int head_dim, int ld_q, int ld_k, int ld_v, int ld_o, float scale, int window, int* status,
-                                     void* stream) {
+                                     int Hkv, int head_dim, int ld_q, int ld_k, int ld_v, int ld_o, float scale, int window, int chunk,
+                                     const void* gate, int ld_gate, int* status, void* stream) {
   if (T <= 0) return 0;
-  return flash_fwd_launch(q, k, v, out, nullptr, cu, n_seq, max_len, 1, T, H, Hkv, head_dim, ld_q, ld_k, ld_v, ld_o, scale, 1, window, status, stream);
+  return flash_fwd_launch(q, k, v, out, nullptr, cu, n_seq, max_len, 1, T, H, Hkv, head_dim, ld_q, ld_k, ld_v, ld_o, scale, 1, window, chunk, gate,
+                          ld_gate, status, stream);
 }

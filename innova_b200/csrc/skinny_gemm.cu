@@ -8,6 +8,7 @@
 // and its tensor-memory set-up and drain cost more than the whole product.)
 //
 // SILU: W holds gate rows [0, N) and up rows [half, half + N); the output is silu(gate) * up.
+// cap > 0 (plain form): the output is cap * tanh(out / cap), the soft limit of logits.
 #include "sm100_common.cuh"
 #include "inv_api.h"
 
@@ -36,7 +37,7 @@ __device__ __forceinline__ uint4 sg_mask(uint4 v, int n) {
 // MT: 16-row tiles of x; NT: 8-column tiles of the CTA (gate tiles when SILU, with as many up tiles behind them).
 template <int MT, int NT, bool SILU>
 __global__ void __launch_bounds__(SG_THREADS) skinny_gemm_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bfloat16* __restrict__ W, int ldw,
-                                                                 int M, int N, int K, int half, void* __restrict__ out, int ldo, int out_f32) {
+                                                                 int M, int N, int K, int half, void* __restrict__ out, int ldo, int out_f32, float cap) {
   constexpr int WT = SILU ? 2 * NT : NT;     // weight tiles
   extern __shared__ float sg_part[];         // [SG_WARPS][MT * 16][WT * 8 + 4]
   constexpr int PL = WT * 8 + 4;
@@ -118,13 +119,15 @@ __global__ void __launch_bounds__(SG_THREADS) skinny_gemm_kernel(const __nv_bflo
       if (SILU) b += sg_part[(size_t)(w * MT * 16 + r) * PL + NT * 8 + c];
     }
     if (SILU) a = a / (1.0f + expf(-a)) * b;
+    else if (cap > 0.f) a = cap * tanhf(a / cap);
     if (out_f32) static_cast<float*>(out)[(size_t)r * ldo + n0 + c] = a;
     else static_cast<__nv_bfloat16*>(out)[(size_t)r * ldo + n0 + c] = __float2bfloat16_rn(a);
   }
 }
 
 template <int MT, int NT, bool SILU>
-static int launch_skinny(const void* x, int ldx, const void* W, int ldw, int M, int N, int K, int half, void* out, int ldo, int out_f32, cudaStream_t st) {
+static int launch_skinny(const void* x, int ldx, const void* W, int ldw, int M, int N, int K, int half, void* out, int ldo, int out_f32, float cap,
+                         cudaStream_t st) {
   constexpr int bytes = SG_WARPS * MT * 16 * ((SILU ? 2 : 1) * NT * 8 + 4) * 4;
   static bool configured = false;
   if (!configured && bytes > 48 * 1024) {
@@ -133,7 +136,7 @@ static int launch_skinny(const void* x, int ldx, const void* W, int ldw, int M, 
   }
   configured = true;
   skinny_gemm_kernel<MT, NT, SILU><<<(N + NT * 8 - 1) / (NT * 8), SG_THREADS, bytes, st>>>((const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, ldw, M, N,
-                                                                                        K, half, out, ldo, out_f32);
+                                                                                        K, half, out, ldo, out_f32, cap);
   const cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
 }
@@ -144,7 +147,7 @@ using namespace inv;
 
 // ldx and ldw are multiples of 8 and at least K rounded up to 8; M <= 64. silu_half > 0: the gated form above.
 extern "C" int inv_skinny_gemm(const void* x, int ldx, const void* W, int ldw, int M, int N, int K, int silu_half, void* out, int ldo, int out_f32,
-                               void* stream) {
+                               float cap, void* stream) {
   const int k8 = (K + 7) & ~7;
   if (M > 64 || (ldx % 8) || (ldw % 8) || ldx < k8 || ldw < k8 || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(W) & 15))
     return -ERR_BAD_ARG;
@@ -152,9 +155,9 @@ extern "C" int inv_skinny_gemm(const void* x, int ldx, const void* W, int ldw, i
   cudaStream_t st = (cudaStream_t)stream;
   const bool wide = N > 148 * 2 * 16;   // enough columns to fill the GPU with 32-column CTAs
 #define INV_SG(MT)                                                                                                                          \
-  (silu_half > 0 ? launch_skinny<MT, 2, true>(x, ldx, W, ldw, M, N, K, silu_half, out, ldo, out_f32, st)                                   \
-   : wide        ? launch_skinny<MT, 4, false>(x, ldx, W, ldw, M, N, K, 0, out, ldo, out_f32, st)                                          \
-                 : launch_skinny<MT, 2, false>(x, ldx, W, ldw, M, N, K, 0, out, ldo, out_f32, st))
+  (silu_half > 0 ? launch_skinny<MT, 2, true>(x, ldx, W, ldw, M, N, K, silu_half, out, ldo, out_f32, cap, st)                                   \
+   : wide        ? launch_skinny<MT, 4, false>(x, ldx, W, ldw, M, N, K, 0, out, ldo, out_f32, cap, st)                                          \
+                 : launch_skinny<MT, 2, false>(x, ldx, W, ldw, M, N, K, 0, out, ldo, out_f32, cap, st))
   if (M <= 16) return INV_SG(1);
   if (M <= 32) return INV_SG(2);
   return INV_SG(4);

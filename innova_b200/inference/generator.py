@@ -170,7 +170,7 @@ class Generator:
         (include/oil/inference_opt.h:262-298). Returns logits [len(tokens), vocab]. The caller truncates the row to the
         part it keeps."""
         if self.stepped:
-            raise NotImplementedError("tree decoding needs a cache that can be rewound; this model keeps recurrent states")
+            raise NotImplementedError("this model has no step over a tree of tokens")
         m, cfg, cache = self.model, self.cfg, self.cache
         T = len(tokens)
         assert 1 <= T <= 64 and all(-1 <= p < i for i, p in enumerate(parents))

@@ -1,28 +1,47 @@
-"""Cache of decoders that mix attention over latents with recurrent layers, and the description of one batch of a step.
+"""Cache of the layer-list decoders, and the description of one batch of a step.
 
-``LatentStateCache`` gives every attention run paged latents (16-token pages, one page table for all runs) and every recurrent
-run a slot per sequence: the delta-rule state in fp32 and the ring of the short convolutions' last inputs. A layer that is
-run several times has one pool or one state per run. Slots follow their sequence when rows are swapped, and need no clearing:
-a sequence that starts at position 0 reads neither. When every attention run has a window, the pages that no window can
-reach any more go back to the pool as the sequence grows.
+``StepCache`` gives every attention run 16-token pages (one page table for all runs) of keys and values, with head counts and sizes
+of its own, or of latents, and every recurrent run a slot per sequence: the delta-rule state in fp32 and the ring of the short
+convolutions' last inputs. A layer that is run several times has one pool or one state per run. Slots follow their sequence when
+rows are swapped, and need no clearing: a sequence that starts at position 0 reads neither. When every attention run has a window
+or a chunked mask, the pages that none of them can reach any more go back to the pool as the sequence grows.
 
 ``StepBatch`` packs the new tokens of several sequences (any number each) into one row of tokens and puts everything the
 kernels need to know about them on the device in one copy."""
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import List, Optional, Sequence
 
 import torch
 
 from ..ops.delta_rule import CHUNK
+from ..ops.kv_attention import first_visible
 from .kv_cache import PAGE, PagedRows
+
+
+@dataclass(frozen=True)
+class KeyValues:
+    """Cache of one attention run: heads and (padded) head size of its keys and values, and the positions it can see."""
+    heads: int
+    dim: int
+    window: Optional[int] = None
+    chunk: Optional[int] = None
+
+
+@dataclass(frozen=True)
+class Latents:
+    """Cache of one attention run over latents of (padded) ``rank`` numbers."""
+    rank: int
+    window: Optional[int] = None
+    chunk: Optional[int] = None
 
 
 class StepBatch:
     """``tokens[i]`` are the next tokens of cache row ``rows[i]``, which holds ``start[i]`` already. ``want``: packed indices
     whose logits are asked for (None: the last token of every sequence)."""
 
-    def __init__(self, cache: "LatentStateCache", tokens: Sequence[Sequence[int]], start: Sequence[int], rows: Sequence[int],
+    def __init__(self, cache: "StepCache", tokens: Sequence[Sequence[int]], start: Sequence[int], rows: Sequence[int],
                  want: Optional[Sequence[int]] = None, vocab: Optional[int] = None):
         lens = [len(t) for t in tokens]
         if not lens or min(lens) < 1:
@@ -73,28 +92,34 @@ class StepBatch:
         self._fill(cache, [int(t) for t in tokens], list(range(self.n + 1)), range(self.n))
 
 
-class LatentStateCache(PagedRows):
-    """``latents``: (padded rank, window or None) per attention run; ``states``: ``DeltaShape`` per recurrent run."""
+class StepCache(PagedRows):
+    """``kv``: ``KeyValues`` per attention run; ``latents``: ``Latents`` per run of attention over latents; ``states``: ``DeltaShape``
+    per recurrent run. ``rewind``: how many of a sequence's last tokens ``truncate`` must be able to drop (their pages are kept)."""
 
-    def __init__(self, latents, states, max_batch: int, max_seq: int, device, dtype=torch.bfloat16, num_pages: Optional[int] = None):
+    def __init__(self, max_batch: int, max_seq: int, device, dtype=torch.bfloat16, num_pages: Optional[int] = None, kv: Sequence[KeyValues] = (),
+                 latents: Sequence[Latents] = (), states: Sequence = ()):
         super().__init__(max_batch, max_seq, device, num_pages)
-        self.windows = [w for _, w in latents]
-        self.dtype = dtype
-        self.latent = [torch.zeros(self.num_pages, PAGE, r, dtype=dtype, device=self.device) for r, _ in latents]
+        self.dtype, self.rewind = dtype, 0
+        self.kv = [torch.zeros(self.num_pages, s.heads, 2, PAGE, s.dim, dtype=dtype, device=self.device) for s in kv]
+        self.latent = [torch.zeros(self.num_pages, PAGE, s.rank, dtype=dtype, device=self.device) for s in latents]
         self.state = [torch.zeros(max_batch, s.H, s.D, s.Dv, dtype=torch.float32, device=self.device) for s in states]
         self.ring = [torch.zeros(max_batch, s.taps, s.channels, dtype=torch.float32, device=self.device) for s in states]
         self._slot = list(range(max_batch))
-        self.reach = None if (not latents or any(not w for w in self.windows)) else max(self.windows)
+        self.masks = sorted({(s.window or 0, s.chunk or 0) for s in (*kv, *latents)})
 
     def slot_of(self, row: int) -> int:
         return self._slot[row]
 
     def bytes_per_token(self) -> int:
-        return sum(p.shape[2] * p.element_size() for p in self.latent)
+        return sum(p.numel() // (self.num_pages * PAGE) * p.element_size() for p in self.kv + self.latent)
 
     def state_bytes(self) -> int:
         """Bytes of one sequence's recurrent states and convolution inputs."""
         return sum(t[0].numel() * 4 for t in self.state + self.ring)
+
+    def first_needed(self, n: int) -> int:
+        """The first cached position that a token at position ``n`` or later sees in any run."""
+        return min((first_visible(n, w, c) for w, c in self.masks), default=0)
 
     def swap(self, a: int, b: int):
         super().swap(a, b)
@@ -104,13 +129,16 @@ class LatentStateCache(PagedRows):
         if new_len == 0:
             self.free(b)
         elif new_len != self._host_lens[b]:
-            raise RuntimeError("a recurrent state cannot be rewound")
+            if self.state:
+                raise RuntimeError("a recurrent state cannot be rewound")
+            if self.first_needed(new_len) < self._released[b] * PAGE or new_len > self._host_lens[b]:
+                raise RuntimeError(f"pages of a sequence of {self._host_lens[b]} tokens that one of {new_len} needs have been given back")
+            super().truncate(b, new_len)
 
     def commit(self, batch_ids: List[int], new_lens: List[int]):
         for b, n in zip(batch_ids, new_lens):
             self._host_lens[b] = n
-            if self.reach is not None:      # the next token sees positions > n - reach
-                self.release_before(b, n - self.reach + 1)
+            self.release_before(b, self.first_needed(max(0, n - self.rewind)))
 
     def free(self, b: int):
         self._free.extend(reversed(self._host_pages[b][self._released[b]:]))

@@ -2,7 +2,8 @@
 
 A module is built for one set of sizes, loads its tensors by name (``load``), gives them back under the same names
 (``export``), and runs on packed tokens (``run(ctx, h, cache_index)``). ``ctx`` is the step (``StepContext``): it chooses the
-projections' precision and kernel.
+projections' precision and kernel. A mixer says what a run of it keeps: ``cache_kind`` (an argument of ``StepCache``) and
+``cache_spec``; ``check`` refuses settings that it does not have.
 
 Weights of the projections are kept in the model's type with rows padded to 16 bytes; everything that enters a norm, a
 convolution, a decay or a residual is fp32."""
@@ -14,10 +15,13 @@ import torch
 import torch.nn as nn
 import torch.nn.functional as F
 
+from ..inference.state_cache import KeyValues, Latents
 from ..ops import delta_rule as dr
+from ..ops import kv_attention as ka
 from ..ops import latent_attention as la
 from ..ops.gemm import EPI_ATOMIC, NUM_SMS, SKINNY_ROWS, gemm, skinny_gemm
 from ..ops.hyper import gated_silu
+from ..ops.sandwich import softcap_
 
 
 def pad_to(n: int, m: int) -> int:
@@ -74,7 +78,95 @@ class StepContext:
         return gated_silu(self.project(x, p), ff, self.dtype)
 
 
-class LatentAttention(nn.Module):
+    def logits(self, h: torch.Tensor, p: Proj, vocab: int, softcap=None) -> torch.Tensor:
+        """fp32 [rows, vocab] of the output head, through the soft limit softcap * tanh(z / softcap) if there is one."""
+        if self.bf16 and h.shape[0] <= SKINNY_ROWS:
+            return skinny_gemm(h[:, : p.k], p.weight[:, : p.k], softcap=softcap or 0.0)[:, :vocab]
+        z = self.project(h, p, torch.float32)[:, :vocab]
+        return softcap_(z, softcap) if softcap else z
+
+
+class Mixer(nn.Module):
+    @classmethod
+    def check(cls, m: dict, layer: int):
+        pass
+
+
+class GatedAttention(Mixer):
+    """Grouped-query attention whose projected keys (before norm and rotation) are the values, with RMS norms over the whole query
+    and key rows, rotary positions on neighbouring pairs of the first dimensions, a mask of chunks counted from position 0, and a
+    sigmoid gate on the output.
+
+    Heads are padded with zero weights to a multiple of 64 in bf16 (the tensor-core kernels' sizes). Whole bf16 prompts run the
+    tcgen05 flash kernel, everything else attends over the pages."""
+
+    kind = "attention"
+    cache_kind = "kv"
+
+    def __init__(self, width: int, m: dict, eps: float, dtype, shapes=None):
+        super().__init__()
+        self.H, self.G, self.D = m["heads"], m["kv_heads"], m["dim"]
+        self.scale, self.eps, self.width = float(m["scale"]), eps, width
+        self.chunk = (m.get("mask") or {}).get("size")
+        self.Dp = pad_to(self.D, 64 if dtype == torch.bfloat16 and self.D <= 256 else 8)
+        self.nq, self.nk = self.H * self.Dp, self.G * self.Dp
+        self.inp = Proj(2 * self.nq + self.nk, width, dtype)         # queries, keys, gate
+        self.q_norm, self.k_norm = frozen(self.nq, dtype=torch.float32), frozen(self.nk, dtype=torch.float32)
+        rot = m.get("rot")
+        self.register_buffer("freq", ka.rope_frequencies(rot["dims"], rot["base"], rot.get("scaling")) if rot else torch.zeros(0), persistent=False)
+        self.out = Proj(width, self.nq, dtype)
+
+    @classmethod
+    def check(cls, m: dict, layer: int):
+        if m["vdim"] != m["dim"]:
+            raise ValueError(f"layer {layer}: values are the keys, but vdim {m['vdim']} is not dim {m['dim']}")
+        if m["heads"] % m["kv_heads"]:
+            raise ValueError(f"layer {layer}: {m['heads']} heads do not share {m['kv_heads']} key heads evenly")
+        rot = m.get("rot")
+        if rot and (rot["dims"] % 2 or not 0 <= rot["dims"] <= m["dim"]):
+            raise ValueError(f"layer {layer}: cannot rotate {rot['dims']} of {m['dim']} dimensions")
+
+    @property
+    def cache_spec(self):
+        return KeyValues(self.G, self.Dp, chunk=self.chunk)
+
+    @torch.no_grad()
+    def load(self, t: Dict[str, torch.Tensor], p: str):
+        H, G, D, Dp, E = self.H, self.G, self.D, self.Dp, self.width
+        for name, off, n in (("q", 0, H), ("k", self.nq, G), ("g", self.nq + self.nk, H)):
+            self.inp.weight.data[off:off + n * Dp].view(n, Dp, -1)[:, :D, :E].copy_(t[p + name].view(n, D, E))
+        self.q_norm.data.view(H, Dp)[:, :D].copy_(t[p + "q.norm"].view(H, D))
+        self.k_norm.data.view(G, Dp)[:, :D].copy_(t[p + "k.norm"].view(G, D))
+        self.out.weight.data[:E, :self.nq].view(E, H, Dp)[:, :, :D].copy_(t[p + "o"].view(E, H, D))
+
+    def export(self, p: str) -> Dict[str, torch.Tensor]:
+        H, G, D, Dp, E = self.H, self.G, self.D, self.Dp, self.width
+        out = {p + name: self.inp.weight[off:off + n * Dp].view(n, Dp, -1)[:, :D, :E].reshape(n * D, E)
+               for name, off, n in (("q", 0, H), ("k", self.nq, G), ("g", self.nq + self.nk, H))}
+        out.update({p + "q.norm": self.q_norm.view(H, Dp)[:, :D].reshape(-1), p + "k.norm": self.k_norm.view(G, Dp)[:, :D].reshape(-1),
+                    p + "o": self.out.weight[:E, :self.nq].view(E, H, Dp)[:, :, :D].reshape(E, H * D)})
+        return out
+
+    @staticmethod
+    def shapes(width: int, m: dict, p: str, ranks) -> Dict[str, tuple]:
+        nq, nk = m["heads"] * m["dim"], m["kv_heads"] * m["dim"]
+        return {p + "q": (nq, width), p + "k": (nk, width), p + "q.norm": (nq,), p + "k.norm": (nk,), p + "g": (nq, width), p + "o": (width, nq)}
+
+    def run(self, ctx: StepContext, h: torch.Tensor, index: int) -> torch.Tensor:
+        b, cache, nq, nk = ctx.batch, ctx.cache, self.nq, self.nk
+        proj = ctx.project(h, self.inp)
+        flash = ctx.bf16 and b.fresh and not b.single and self.Dp <= 128
+        q, k = ka.qkv_append(proj, 0, nq, nq, self.H, self.G, self.D, self.Dp, self.q_norm, self.k_norm, self.eps, self.freq, cache.kv[index],
+                             cache.page_table, b, want_k=flash)
+        gate = proj[:, nq + nk:2 * nq + nk]
+        if flash:
+            o = la.packed_flash(q, k, proj[:, nq:nq + nk], self.H, self.Dp, self.scale, None, b, kv_heads=self.G, chunk=self.chunk, gate=gate)
+        else:
+            o = ka.kv_attend(q, cache.kv[index], cache.page_table, self.H, self.scale, b, chunk=self.chunk, gate=gate)
+        return ctx.project(o, self.out)
+
+
+class LatentAttention(Mixer):
     """Attention whose keys and values are linear images of one cached latent per token, optionally windowed.
 
     Query / value heads are padded to ``Dp`` (64 or 128 where they fit, for the tcgen05 flash kernel) and the latent to ``Rp``
@@ -82,6 +174,7 @@ class LatentAttention(nn.Module):
     prompt and 32-bit models attend in the latent space."""
 
     kind = "latent_attention"
+    cache_kind = "latents"
 
     def __init__(self, width: int, m: dict, eps: float, dtype, shapes=None):
         super().__init__()
@@ -99,8 +192,8 @@ class LatentAttention(nn.Module):
         self.out = Proj(width, self.off_c, dtype)
 
     @property
-    def latent(self):
-        return self.Rp, self.window
+    def cache_spec(self):
+        return Latents(self.Rp, window=self.window)
 
     @torch.no_grad()
     def load(self, t: Dict[str, torch.Tensor], p: str):
@@ -146,10 +239,11 @@ class LatentAttention(nn.Module):
         return ctx.project(o, self.out)
 
 
-class ChannelDelta(nn.Module):
+class ChannelDelta(Mixer):
     """Gated delta rule with short convolutions, a low-rank decay per key channel and a low-rank output gate."""
 
     kind = "channel_delta"
+    cache_kind = "states"
 
     def __init__(self, width: int, m: dict, eps: float, dtype, shapes=None):
         super().__init__()
@@ -163,6 +257,10 @@ class ChannelDelta(nn.Module):
         self.A_log, self.dt_bias = frozen(s.H, dtype=torch.float32), frozen(s.H * s.D, dtype=torch.float32)
         self.norm = frozen(s.Dv, dtype=torch.float32)
         self.out = Proj(width, s.H * s.Dv, dtype)
+
+    @property
+    def cache_spec(self):
+        return self.shape
 
     @torch.no_grad()
     def load(self, t: Dict[str, torch.Tensor], p: str):
@@ -237,4 +335,4 @@ class GatedMLP(nn.Module):
         return ctx.project(ctx.gated(h, self.inp, self.ff), self.out)
 
 
-MIXERS = {c.kind: c for c in (LatentAttention, ChannelDelta)}
+MIXERS = {c.kind: c for c in (GatedAttention, LatentAttention, ChannelDelta)}

@@ -19,7 +19,7 @@ def register(name: str):
 
 def model_class(config: dict) -> type:
     """The registered model class of a configuration dictionary."""
-    from . import vebesun  # noqa: F401  (registers itself)
+    from . import mekazen, vebesun  # noqa: F401  (they register themselves)
     name = config.get("architecture")
     if name not in ARCHITECTURES:
         raise ValueError(f"unknown architecture {name!r}; known: {', '.join(sorted(ARCHITECTURES))}")

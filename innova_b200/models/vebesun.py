@@ -3,10 +3,7 @@
 The residual is a bundle of streams joined by hyper-connections (``ops/hyper.py``), norms are LayerNorm in front of every
 sublayer, a stretch of layers can be run several times with the same weights (each pass with a cache of its own), positions
 enter through the mixers only, and the output head is the embedding table. Mixers: windowed latent attention and the
-channel-wise gated delta rule (``models/mixers.py``).
-
-The model has one forward: ``step(cache, batch)`` runs the packed new tokens of any number of sequences against a
-``LatentStateCache`` and returns the logits asked for. Generation, batching, scoring and trace replay all go through it."""
+channel-wise gated delta rule (``models/mixers.py``); weights, cache and step are those of ``models/stepped.py``."""
 from __future__ import annotations
 
 from dataclasses import dataclass, field
@@ -15,11 +12,10 @@ from typing import Dict, List, Optional, Tuple
 import torch
 import torch.nn as nn
 
-from ..inference.state_cache import LatentStateCache, StepBatch
-from ..ops.gemm import full_fp32_matmul
 from ..ops.hyper import HyperIn, HyperOut, hyper_step
-from .mixers import MIXERS, GatedMLP, Proj, StepContext, frozen, put
+from .mixers import MIXERS, Proj, StepContext, frozen, put
 from .registry import register
+from .stepped import SteppedDecoder, check_layers, layer_bodies, mlp_shapes
 
 
 @dataclass
@@ -51,11 +47,7 @@ class VebesunConfig:
     def order(self) -> List[int]:
         """Layer index of every run."""
         n = len(self.layers)
-        for i, layer in enumerate(self.layers):
-            if layer["type"] not in MIXERS:
-                raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
-            if layer.get("mlp") is not None and layer["mlp"].get("kind") != "dense":
-                raise ValueError(f"layer {i}: unknown feed-forward {layer['mlp']!r}")
+        check_layers(self.layers)
         if not self.loop:
             return list(range(n))
         a, b, times = self.loop["start"], self.loop["stop"], self.loop["times"]
@@ -79,9 +71,7 @@ class VebesunConfig:
             l = f"l{i}."
             out.update(MIXERS[layer["type"]].shapes(E, layer["mixer"], l + "mix.", self.ranks.get(str(i))))
             if layer.get("mlp") is not None:
-                F = layer["mlp"]["ff"]
-                out[l + "mlp.gate"] = out[l + "mlp.up"] = (F, E)
-                out[l + "mlp.down"] = (E, F)
+                out.update(mlp_shapes(E, layer["mlp"], l + "mlp."))
             for q in ((1, 2) if layer.get("mlp") is not None else (1,)):
                 out[f"{l}norm{q}"] = out[f"{l}norm{q}.b"] = (E,)
                 out[f"{l}hc{q}.in"] = out[f"{l}hc{q}.out"] = (S,)
@@ -101,18 +91,14 @@ class Sublayer(nn.Module):
 
 
 @register("Vebesun")
-class VebesunModel(nn.Module):
+class VebesunModel(SteppedDecoder):
     # what a fresh checkout compiles to run this model
     CUDA_SOURCES = ("hyper.cu", "delta_rule.cu", "latent_attn.cu", "skinny_gemm.cu", "flash_attn_fwd.cu", "gemm_tcgen05.cu", "gemm_tcgen05_2cta.cu", "elementwise.cu",
                     "sampler.cu")
-    HOST_SOURCES = ("importers.cpp",)
     config_class = VebesunConfig
 
     def __init__(self, cfg: VebesunConfig, dtype=torch.bfloat16, device=None, seed: Optional[int] = None):
-        super().__init__()
-        if dtype not in (torch.bfloat16, torch.float32):
-            raise ValueError(f"{dtype}: bfloat16 or float32")
-        self.cfg, self.dtype = cfg, dtype
+        super().__init__(cfg, dtype)
         E, S = cfg.width, cfg.streams
         self.embed = Proj(cfg.vocab_size, E, dtype)
         self.final_w, self.final_b = frozen(E, dtype=torch.float32), frozen(E, dtype=torch.float32)
@@ -120,17 +106,9 @@ class VebesunModel(nn.Module):
         layers = []
         for i, layer in enumerate(cfg.layers):
             sh = {"a1": (cfg.ranks[str(i)][0],), "g1": (cfg.ranks[str(i)][1],)} if str(i) in cfg.ranks else None
-            subs = [Sublayer(MIXERS[layer["type"]](E, layer["mixer"], cfg.norm_eps, dtype, sh), E, S)]
-            if layer.get("mlp") is not None:
-                subs.append(Sublayer(GatedMLP(E, layer["mlp"]["ff"], dtype), E, S))
-            layers.append(nn.ModuleList(subs))
+            layers.append(nn.ModuleList(Sublayer(body, E, S) for body in layer_bodies(E, layer, cfg.norm_eps, dtype, sh)))
         self.layers = nn.ModuleList(layers)
-        # cache index of every run: attention and recurrent runs are counted separately
-        self.runs, counts = [], {}
-        for i in cfg.order():
-            kind = cfg.layers[i]["type"]
-            self.runs.append((i, counts.setdefault(kind, 0)))
-            counts[kind] += 1
+        self.set_runs(cfg.order())
         if seed is not None:
             self.reset_parameters(seed)
         if device is not None:
@@ -143,29 +121,18 @@ class VebesunModel(nn.Module):
         return {str(i): (shapes[f"l{i}.mix.a1"][0], shapes[f"l{i}.mix.g1"][0]) for i in range(len(cfg.layers)) if f"l{i}.mix.a1" in shapes}
 
     @classmethod
-    def from_tensors(cls, config: dict, tensors: Dict[str, torch.Tensor], dtype=torch.bfloat16, device=None) -> "VebesunModel":
-        cfg = VebesunConfig.from_dict(config)
-        cfg.ranks = cls.ranks_from({n: tuple(t.shape) for n, t in tensors.items()}, cfg) or cfg.ranks
-        model = cls(cfg, dtype=dtype)
-        model.load_tensors(tensors)
-        return model.to(device) if device is not None else model
+    def fit_config(cls, cfg: VebesunConfig, shapes: Dict[str, tuple]):
+        cfg.ranks = cls.ranks_from(shapes, cfg) or cfg.ranks
 
-    @torch.no_grad()
-    def load_tensors(self, tensors: Dict[str, torch.Tensor]):
-        shapes = self.cfg.tensor_shapes()
+    def complete(self, tensors, shapes):
         if self.cfg.streams == 1:      # a model with a plain residual has no stream weights: they are ones
             tensors = dict(tensors)
             for n in shapes:
                 if ".hc" in n and n not in tensors:
                     tensors[n] = torch.ones(shapes[n])
-        missing = [n for n in shapes if n not in tensors]
-        if missing:
-            raise KeyError(f"model file lacks {len(missing)} tensors: {', '.join(missing[:8])}")
-        t = {}
-        for n, shp in shapes.items():
-            if tensors[n].numel() != torch.Size(shp).numel():
-                raise ValueError(f"{n}: shape {tuple(tensors[n].shape)}, expected {shp}")
-            t[n] = tensors[n].view(shp)
+        return tensors
+
+    def put_tensors(self, t: Dict[str, torch.Tensor]):
         put(self.embed, t["embed"])
         self.final_w.copy_(t["final.norm"])
         self.final_b.copy_(t["final.norm.b"])
@@ -210,27 +177,6 @@ class VebesunModel(nn.Module):
                 t[n] = torch.randn(shp, generator=g) * shp[-1] ** -0.5
         self.load_tensors(t)
 
-    def num_params(self) -> int:
-        return sum(torch.Size(s).numel() for s in self.cfg.tensor_shapes().values())
-
-    # ------------------------------------------------------------------ cache and step
-    def make_cache(self, max_batch: int, max_seq: int, device=None, num_pages: Optional[int] = None) -> LatentStateCache:
-        latents, states = [], []
-        for i, _ in self.runs:
-            body = self.layers[i][0].body
-            if hasattr(body, "latent"):
-                latents.append(body.latent)
-            else:
-                states.append(body.shape)
-        return LatentStateCache(latents, states, max_batch, max_seq, device or self.embed.weight.device, self.dtype, num_pages)
-
-    @torch.no_grad()
-    def step(self, cache: LatentStateCache, batch: StepBatch, hidden: bool = False, residuals: Optional[list] = None):
-        """Run the batch's new tokens; returns fp32 logits [wanted, vocab] (or the final normed states with ``hidden``), None when
-        nothing is wanted. ``residuals`` collects the sum of the streams after every layer run."""
-        with full_fp32_matmul(self.dtype):
-            return self._step(cache, batch, hidden, residuals)
-
     def _step(self, cache, batch, hidden, residuals):
         cfg = self.cfg
         ctx = StepContext(self, cache, batch)
@@ -258,20 +204,4 @@ class VebesunModel(nn.Module):
             residuals.append(x.sum(1))
         if hidden:
             return h
-        return ctx.project(h, self.embed, torch.float32)[:, : cfg.vocab_size]
-
-    # ------------------------------------------------------------------ whole-sequence forms (scoring, embedding, beam search)
-    def _whole(self, ids: torch.Tensor, hidden: bool):
-        B, S = ids.shape
-        cache = self.make_cache(B, S, self.embed.weight.device)
-        for b in range(B):
-            cache.reserve(b, S)
-        batch = StepBatch(cache, ids.tolist(), [0] * B, list(range(B)), want=range(B * S), vocab=self.cfg.vocab_size)
-        return self.step(cache, batch, hidden=hidden).view(B, S, -1)
-
-    def hidden_states(self, ids: torch.Tensor) -> torch.Tensor:
-        return self._whole(ids, True)
-
-    def forward(self, ids: torch.Tensor) -> torch.Tensor:
-        """[B, S] token ids -> logits [B, S, vocab]."""
-        return self._whole(ids, False)
+        return ctx.logits(h, self.embed, cfg.vocab_size)

@@ -100,19 +100,20 @@ def gemm(a, b, out=None, *, a_mn=False, b_mn=False, M=None, N=None, K=None, epil
     return out
 
 
-_native.register_cuda_sigs({"inv_skinny_gemm": [_native.vp, _native.i32, _native.vp] + [_native.i32] * 5 + [_native.vp, _native.i32, _native.i32, _native.vp]})
+_native.register_cuda_sigs({"inv_skinny_gemm": [_native.vp, _native.i32, _native.vp] + [_native.i32] * 5 +
+                                [_native.vp, _native.i32, _native.i32, _native.f32, _native.vp]})
 SKINNY_ROWS = 32          # the kernel takes 64; beyond 32 the split-K tiled product is faster
 
 
-def skinny_gemm(x, w, n=None, silu_half: int = 0, out_dtype=torch.float32):
+def skinny_gemm(x, w, n=None, silu_half: int = 0, out_dtype=torch.float32, softcap: float = 0.0):
     """x [M <= 64, K] times w [N, K]^T for decode steps (csrc/skinny_gemm.cu): weights straight from memory into MMA fragments,
     no tile set-up. Rows of both operands start on 16-byte boundaries. ``silu_half``: w holds gate rows [0, n) and up rows
-    [silu_half, silu_half + n) and the result is silu(gate) * up."""
+    [silu_half, silu_half + n) and the result is silu(gate) * up. ``softcap``: the result is softcap * tanh(result / softcap)."""
     M, K = x.shape
     n = w.shape[0] if n is None else n
     out = torch.empty((M, (n + 7) // 8 * 8), dtype=out_dtype, device=x.device)
     rt.check(rt.lib().inv_skinny_gemm(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), M, n, K, silu_half, out.data_ptr(), out.stride(0),
-                                      int(out_dtype == torch.float32), rt.stream_ptr()), "inv_skinny_gemm")
+                                      int(out_dtype == torch.float32), float(softcap), rt.stream_ptr()), "inv_skinny_gemm")
     return out[:, :n]
 
 

@@ -17,7 +17,7 @@ _native.register_cuda_sigs({
     "inv_latent_prep": [_vp, _i, _i, _i, _i, _i, _vp, _f, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _vp],
     "inv_head_proj": [_vp, _i, _i, _vp, _i, _i, _i, _vp, _i, _i, _i, _vp],
     "inv_latent_attend": [_vp, _vp, _i, _i, _vp, _i, _vp, _vp, _vp, _i, _f, _vp, _vp, _i, _i, _i, _vp],
-    "inv_flash_attn_packed": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _vp],
+    "inv_flash_attn_packed": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _i, _vp, _vp],
 })
 
 PAGE = 16
@@ -85,11 +85,15 @@ def latent_attend(q: torch.Tensor, pool, page_table, heads: int, scale: float, w
     return out
 
 
-def packed_flash(q, k, v, heads: int, head_dim: int, scale: float, window: Optional[int], batch) -> torch.Tensor:
-    """Causal (windowed) flash attention of packed whole prompts; q, k, v [T, heads * head_dim] row views, head_dim 64 or 128."""
+def packed_flash(q, k, v, heads: int, head_dim: int, scale: float, window: Optional[int], batch, kv_heads: Optional[int] = None,
+                 chunk: Optional[int] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal flash attention of packed whole prompts, windowed or chunked; q [T, heads * head_dim], k and v [T, kv_heads * head_dim]
+    (default: as many as query heads) row views, head_dim 64 or 128. ``gate`` [T, heads * head_dim] bf16: the result is multiplied
+    by its sigmoid."""
     T = q.shape[0]
     out = torch.empty(T, heads * head_dim, dtype=torch.bfloat16, device=q.device)
     rt.check(rt.lib().inv_flash_attn_packed(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), batch.cu.data_ptr(), batch.n, T, batch.max_len,
-                                            heads, heads, head_dim, q.stride(0), k.stride(0), v.stride(0), out.stride(0), float(scale),
-                                            int(window or 0), rt.status_tensor(q.device).data_ptr(), rt.stream_ptr()), "inv_flash_attn_packed")
+                                            heads, kv_heads or heads, head_dim, q.stride(0), k.stride(0), v.stride(0), out.stride(0), float(scale),
+                                            int(window or 0), int(chunk or 0), rt.ptr(gate), 0 if gate is None else gate.stride(0),
+                                            rt.status_tensor(q.device).data_ptr(), rt.stream_ptr()), "inv_flash_attn_packed")
     return out

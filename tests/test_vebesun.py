@@ -4,9 +4,6 @@ Every test makes its own small configuration and seeded weights. The ``dev`` fix
 box, on the CUDA kernels in 32-bit and in bf16 (``cuda-f32``, ``cuda-bf16``)."""
 import json
 import math
-import os
-import subprocess
-import sys
 
 import numpy as np
 import pytest
@@ -14,15 +11,12 @@ import torch
 
 import vebesun_oracle as oracle
 from innova_b200.inference.generator import Generator
-from innova_b200.inference.state_cache import LatentStateCache, StepBatch
+from innova_b200.inference.state_cache import Latents, StepBatch, StepCache
 from innova_b200.models.vebesun import VebesunConfig, VebesunModel
 from innova_b200.ops import delta_rule as dr
 from innova_b200.ops import latent_attention as la
 from innova_b200.ops.hyper import HyperIn, HyperOut, gated_silu, hyper_step
-
-ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-BOTH = [("cpu", torch.float32), pytest.param(("cuda", torch.float32), marks=pytest.mark.gpu), pytest.param(("cuda", torch.bfloat16), marks=pytest.mark.gpu)]
-IDS = ["cpu-f32", "cuda-f32", "cuda-bf16"]
+from stepped_util import BOTH, IDS, error, replay, run, tokens, tol, with_config, write_dir
 
 
 @pytest.fixture(params=BOTH, ids=IDS)
@@ -67,33 +61,6 @@ CONFIGS = {
 def build(cfg, dev, seed=0, **kw):
     w = oracle.random_weights(cfg, seed, **kw)
     return VebesunModel.from_tensors(cfg, w, dtype=dev[1], device=dev[0]), w
-
-
-def tokens(n, cfg, seed):
-    return torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
-
-
-def error(got, want):
-    """Root mean square of the difference over the logits' own, worst row."""
-    d = got.double().cpu() - want
-    return float((d.square().mean(-1).sqrt() / want.square().mean(-1).sqrt().clamp_min(1e-6)).max())
-
-
-def tol(dev):
-    return 6e-2 if dev[1] == torch.bfloat16 else 3e-5
-
-
-def run(model, toks, cuts, cache=None, row=0):
-    """Logits of every position when the sequence arrives in portions of the given sizes (the last size repeats)."""
-    cache = cache or model.make_cache(2, len(toks) + 1)
-    out, pos, k = [], 0, 0
-    while pos < len(toks):
-        n = min(cuts[min(k, len(cuts) - 1)], len(toks) - pos)
-        cache.reserve(row, pos + n)
-        out.append(model.step(cache, StepBatch(cache, [toks[pos:pos + n]], [pos], [row], want=range(n), vocab=model.cfg.vocab_size)))
-        pos, k = pos + n, k + 1
-        cache.commit([row], [pos])
-    return torch.cat(out)
 
 
 # ------------------------------------------------------------------------------------------------ mechanisms alone
@@ -159,7 +126,7 @@ class Rows:
     """Cache rows for a mechanism on its own: rings and states of one recurrent run, or pages of one attention run."""
 
     def __init__(self, d, dt, states=(), latents=(), n=4, max_seq=512):
-        self.c = LatentStateCache(list(latents), list(states), n, max_seq, d, dt)
+        self.c = StepCache(n, max_seq, d, dt, latents=latents, states=states)
 
     def batch(self, lens, start, rows):
         for r, n, s in zip(rows, lens, start):
@@ -274,7 +241,7 @@ def test_latent_attention_sees_exactly_its_window(dev, H, R, window):
     far = [0, 15, 16, 31, 59, 60, 61, 127, 128, 255, 256]
     c[far] += 9.0 * dirs[torch.arange(len(far)) % H]            # the key each head looks for
     c = c.to(dt)
-    rc = Rows(d, dt, latents=[((R + 15) // 16 * 16, window)])
+    rc = Rows(d, dt, latents=[Latents((R + 15) // 16 * 16, window)])
     b = rc.batch([n], [0], [1])
     nw = torch.ones(R, device=d)
     la.latent_append(c.to(d), 0, R, nw, 0.0, rc.c.latent[0], rc.c.page_table, b)
@@ -307,7 +274,7 @@ def test_head_products(T, K, N):
 def test_packed_flash_attention(D, window):
     lens, H = [1, 300, 129, 128, 64], 3
     q, k, v = (torch.randn(sum(lens), H * D, device="cuda").bfloat16() for _ in range(3))
-    rc = Rows("cuda", torch.bfloat16, latents=[(16, window)], n=5)
+    rc = Rows("cuda", torch.bfloat16, latents=[Latents(16, window)], n=5)
     got = la.packed_flash(q, k, v, H, D, D ** -0.5, window, rc.batch(lens, [0] * 5, range(5))).float()
     at = 0
     for n in lens:
@@ -527,18 +494,6 @@ def test_decode_graphs_equal_eager_steps():
         assert list(gen._graphs) == [3]
 
 
-def write_dir(path, cfg, w):
-    path.mkdir()
-    (path / "config.json").write_text(json.dumps(cfg))
-    head, blob = {}, b""
-    for n, t in w.items():
-        raw = t.bfloat16().contiguous().view(torch.int16).numpy().tobytes()
-        head[n] = {"dtype": "BF16", "shape": list(t.shape), "data_offsets": [len(blob), len(blob) + len(raw)]}
-        blob += raw
-    js = json.dumps(head).encode()
-    (path / "model.safetensors").write_bytes(len(js).to_bytes(8, "little") + js + blob)
-
-
 def test_model_directory_and_oil_file(tmp_path):
     from innova_b200.formats import export
     cfg = CONFIGS["odd"]
@@ -557,13 +512,7 @@ def test_model_directory_and_oil_file(tmp_path):
     with pytest.raises(KeyError, match="l1.mix.norm"):
         export.load_model(str(tmp_path / "bad"))
     with pytest.raises(ValueError, match="architecture"):
-        export.load_model_dir(_with_config(tmp_path, {"architecture": "nothing"}))
-
-
-def _with_config(tmp_path, cfg):
-    (tmp_path / "c").mkdir()
-    (tmp_path / "c" / "config.json").write_text(json.dumps(cfg))
-    return str(tmp_path / "c")
+        export.load_model_dir(with_config(tmp_path, {"architecture": "nothing"}))
 
 
 def test_configuration():
@@ -575,14 +524,6 @@ def test_configuration():
         VebesunConfig.from_dict({**CONFIGS["mixed"], "loop": {"start": 2, "stop": 9, "times": 2}})
     with pytest.raises(ValueError):
         VebesunConfig.from_dict(config([{"type": "other", "mixer": {}, "mlp": None}]))
-
-
-def replay(model_dir, out, steps, dtype, device):
-    out.mkdir()
-    r = subprocess.run([sys.executable, os.path.join(ROOT, "bin", "trace_run"), "--model", str(model_dir), "--dtype", dtype, "--out", str(out),
-                        "--max-tokens", "512", "--device", device], input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True)
-    assert r.returncode == 0, r.stderr
-    assert [x for x in r.stdout.splitlines() if x.startswith("done")] == [f"done {s['step']}" for s in steps]
 
 
 def test_trace_replay(dev, tmp_path):
