@@ -89,8 +89,8 @@ def parse():
     ap.add_argument("--engine", default="fsdp3", choices=["fsdp3", "zero2"], help="data-parallel engine at N > 1")
     ap.add_argument("--decode-new", type=int, default=64, help="generated tokens of the decode section (0: skip it)")
     ap.add_argument("--decode-layers", type=int, default=32, help="for debugging only; the reported decode config is 32")
-    ap.add_argument("--design", default=None, choices=["vebesun"], help="instead of the headline workload: throughput of one model design "
-                    "beside the closest models at equal size (bench_vebesun.py)")
+    ap.add_argument("--design", default=None, choices=["vebesun", "mekazen"], help="instead of the headline workload: throughput of one model design "
+                    "beside the closest models at equal size (bench_<design>.py)")
     ap.add_argument("--section", default="all", choices=["all", "model", "kernels"], help="with --design: what to measure")
     ap.add_argument("--sizes", default="", help="with --design: sizes to measure, with commas")
     return ap.parse_args()
@@ -332,9 +332,9 @@ def run_ours(args):
 
 def main():
     args = parse()
-    if args.design == "vebesun":
-        import bench_vebesun
-        return bench_vebesun.main(args.section, args.sizes.split(",") if args.sizes else None)
+    if args.design:
+        import importlib
+        return importlib.import_module(f"bench_{args.design}").main(args.section, args.sizes.split(",") if args.sizes else None)
     if args.impl == "reference":
         return run_reference(args)
     run_ours(args)

@@ -7,10 +7,9 @@ Closest models: ``HybridEngine`` (the other gated delta-rule decoder; one sequen
 model figures run over weights larger than L2, the kernel figures flush L2 before every call."""
 from __future__ import annotations
 
-import json
-import os
-
 import torch
+
+from bench_design import KernelBench, emit, timed
 
 SIZES = {
     # name: width, ff, heads (head size 128), latent rank, vocabulary
@@ -19,15 +18,6 @@ SIZES = {
     "4k": (4096, 11008, 32, 512, 32768),
 }
 WINDOW, LAYERS, STREAMS, RANK = 1024, 8, 4, 128
-
-
-def peaks():
-    path = os.path.join(os.path.dirname(os.path.abspath(__file__)), "MEASURED_PEAKS.json")
-    if os.path.exists(path):
-        with open(path) as f:
-            p = json.load(f)
-        return p["hbm_gbs"], p["bf16_tflops"], "measured"
-    return 6650.0, 1590.0, "fallback"
 
 
 def vebesun_config(size):
@@ -39,23 +29,6 @@ def vebesun_config(size):
     layers = [attn if i % 4 == 3 else delta for i in range(LAYERS)]
     ranks = {str(i): (RANK, RANK) for i in range(LAYERS) if i % 4 != 3}
     return VebesunConfig(vocab_size=V, width=E, layers=layers, streams=STREAMS, embedding_scale=E ** 0.5, max_seq_len=8192 + 64, ranks=ranks)
-
-
-def timed(fn, reps, warm=3):
-    for _ in range(warm):
-        fn()
-    torch.cuda.synchronize()
-    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-    e0.record()
-    for _ in range(reps):
-        fn()
-    e1.record()
-    torch.cuda.synchronize()
-    return e0.elapsed_time(e1) / reps
-
-
-def emit(**kw):
-    print(json.dumps(kw), flush=True)
 
 
 def model_section(sizes):
@@ -153,28 +126,8 @@ def kernel_section(size="2k"):
     from innova_b200.ops.hyper import HyperIn, HyperOut, gated_silu, hyper_step
     E, F, H, R, V = SIZES[size]
     dev, bf = torch.device("cuda"), torch.bfloat16
-    hbm, tf, src = peaks()
-    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
-    fp32_tf = 148 * 128 * 2 * 1.965e9 / 1e12          # one fp32 FMA per lane and clock at the maximum clock
-
-    def cold(fn, reps=8):
-        for _ in range(3):
-            fn()
-        ms = []
-        for _ in range(reps):
-            flush.add_(1)
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            e0.record()
-            fn()
-            e1.record()
-            torch.cuda.synchronize()
-            ms.append(e0.elapsed_time(e1))
-        return sorted(ms)[len(ms) // 2]
-
-    def report(name, shape, ms, gbytes=0.0, tflop=0.0, fp32=0.0, like=None):
-        t = {"hbm": gbytes / hbm * 1e3, "bf16": tflop / tf * 1e3, "fp32": fp32 / fp32_tf * 1e3}
-        bound = max(t, key=t.get)
-        emit(metric="kernel", kernel=name, shape=shape, us=ms * 1e3, bound=bound, roofline_us=t[bound] * 1e3, fraction=t[bound] / ms, peaks=src, like=like)
+    bench = KernelBench(dev)
+    cold, report = bench.cold, bench.report
     rand = lambda *s: torch.randn(*s, device=dev)
     # residual step (streams) and, as the like kernel, the fused residual-add RMSNorm of the dense decoder
     for T in (8192, 64):

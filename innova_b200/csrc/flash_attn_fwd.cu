@@ -32,8 +32,8 @@ struct FlashFwdParams {
   float scale;
   int causal;
   int window;  // > 0 (causal only): a query sees the `window` most recent keys, its own position included
-  int chunk;   // > 0 (causal only): a query sees the earlier keys of its own chunk of `chunk` positions (counted from position 0)
-  const __nv_bfloat16* gate;  // the output is multiplied by sigmoid(gate), element by element; null: no gate
+  int chunk;   // EXT; > 0 (causal only): a query sees the earlier keys of its own chunk of `chunk` positions (counted from position 0)
+  const __nv_bfloat16* gate;  // EXT: the output is multiplied by sigmoid(gate), element by element; null: no gate
   int ld_gate;
   const int* cu;  // packed batch: sequence b is rows [cu[b], cu[b + 1]) of the token-major buffers; null: B sequences of S rows
   int* status;
@@ -63,7 +63,8 @@ struct Fwd3Smem {
   static constexpr int TOTAL = BAR_OFF + 256 + 1024;
 };
 
-template <int ND>
+// EXT: with the chunked mask and the output gate (registers the plain form does not spend).
+template <int ND, bool EXT>
 __global__ void __launch_bounds__(FA_THREADS, ND == 1 ? 2 : 1)
 flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                   const __grid_constant__ CUtensorMap tmap_v, const FlashFwdParams p) {
@@ -98,7 +99,7 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
   const int nkb_all = (S + FA_BN - 1) / FA_BN;
   // key blocks visited: [jlo, jlo + nkb). A sliding window skips the blocks that lie wholly before the first query's window, a
   // chunked mask those before the first query's chunk.
-  const int jlo = !p.causal ? 0 : p.window > 0 ? max(0, q0 - p.window + 1) / FA_BN : p.chunk > 0 ? (q0 - q0 % p.chunk) / FA_BN : 0;
+  const int jlo = !p.causal ? 0 : p.window > 0 ? max(0, q0 - p.window + 1) / FA_BN : EXT && p.chunk > 0 ? (q0 - q0 % p.chunk) / FA_BN : 0;
   const int nkb = (p.causal ? min(nkb_all, q_blk + 1) : nkb_all) - jlo;
   constexpr uint32_t TMEM_COLS = ND == 1 ? 256 : 512;
   constexpr uint32_t O_COL = 128, P_COL = 128 + D;
@@ -191,17 +192,17 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     const uint32_t t_lane = tmem_base + (uint32_t(q * 32) << 16);
     const float c = p.scale * 1.4426950408889634f;
     float m_used = -INFINITY, l = 0.f;
-    const bool windowed = p.causal && p.window > 0, chunked = p.causal && p.chunk > 0;
-    const int kmin = windowed ? row - p.window + 1 : chunked ? row - row % p.chunk : 0;
-    const int last = min(q0 + FA_BM, S) - 1;                    // the block's last row has the highest first visible key
-    const int kmin_last = windowed ? last - p.window + 1 : chunked ? last - last % p.chunk : 0;
     bool ok = true;
     for (int j = 0; j < nkb; ++j) {
       if (!mbar_wait_warp(s_full, j & 1, abort_flag, p.status, ERR_WAIT_TMEM_FULL)) { ok = false; break; }
       tc_fence_after();
       const int k0 = (jlo + j) * FA_BN;
-      const bool need_mask = (p.causal && k0 + FA_BN - 1 > q0) || (k0 + FA_BN > S) || k0 < kmin_last;
+      const bool windowed = p.causal && p.window > 0, chunked = EXT && p.causal && p.chunk > 0;
+      const int last = q0 + FA_BM - 1;           // the block's last row has the highest first visible key
+      const bool need_mask = (p.causal && k0 + FA_BN - 1 > q0) || (k0 + FA_BN > S) || (windowed && k0 <= last - p.window) ||
+                             (chunked && k0 < last - last % p.chunk);
       const int kmax = p.causal ? min(row, S - 1) : S - 1;
+      const int kmin = windowed ? row - p.window + 1 : chunked ? row - row % p.chunk : 0;
       uint32_t sr[128];
       tmem_ld_32x32(t_lane, sr);
       tmem_ld_32x32(t_lane + 32, sr + 32);
@@ -266,24 +267,30 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       __syncwarp();
       if (lane == 0) mbar_arrive(p_full);
     }
+    const size_t grow = (p.cu ? (size_t)row_base : (size_t)b * S) + row;
+    uint4 gv[EXT ? D / 8 : 1];                    // the row's gate, requested while the last PV MMA runs
+    const bool gated = EXT && p.gate != nullptr;
+    if (gated && row < S) {
+      const __nv_bfloat16* gate = p.gate + grow * p.ld_gate + h * D;
+#pragma unroll
+      for (int i = 0; i < (EXT ? D / 8 : 1); ++i) gv[i] = *reinterpret_cast<const uint4*>(gate + i * 8);
+    }
     if (ok) ok = mbar_wait_warp(o_full, (nkb - 1) & 1, abort_flag, p.status, ERR_WAIT_TMEM_FULL);
     if (ok) {
       tc_fence_after();
       const float inv_l = l > 0.f ? 1.f / l : 0.f;
-      const size_t grow = (p.cu ? (size_t)row_base : (size_t)b * S) + row;
       __nv_bfloat16* dst = p.out + grow * p.ld_o + h * D;
-      const __nv_bfloat16* gate = p.gate ? p.gate + grow * p.ld_gate + h * D : nullptr;
-#pragma unroll 1
+#pragma unroll (EXT ? D / 32 : 1)
       for (int cc = 0; cc < D / 32; ++cc) {
         uint32_t rr[32];
         tmem_ld_32x32(t_lane + O_COL + cc * 32, rr);
         tmem_ld_wait();
         if (row < S) {
-          if (gate) {
+          if (gated) {
 #pragma unroll
             for (int g = 0; g < 4; ++g) {
-              const uint4 gv = *reinterpret_cast<const uint4*>(gate + cc * 32 + g * 8);
-              const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w};
+              const uint4 g4 = gv[EXT ? cc * 4 + g : 0];
+              const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
 #pragma unroll
               for (int i = 0; i < 4; ++i) {
                 const float g0 = __uint_as_float(gw[i] << 16), g1 = __uint_as_float(gw[i] & 0xffff0000u);
@@ -387,12 +394,17 @@ static int flash_fwd_launch(const void* q, const void* k, const void* v, void* o
   cudaStream_t st = (cudaStream_t)stream;
   static bool configured = false;
   if (!configured) {
-    cudaFuncSetAttribute(flash_fwd3_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, Fwd3Smem<1>::TOTAL);
-    cudaFuncSetAttribute(flash_fwd3_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, Fwd3Smem<2>::TOTAL);
+    cudaFuncSetAttribute(flash_fwd3_kernel<1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, Fwd3Smem<1>::TOTAL);
+    cudaFuncSetAttribute(flash_fwd3_kernel<2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, Fwd3Smem<2>::TOTAL);
+    cudaFuncSetAttribute(flash_fwd3_kernel<1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, Fwd3Smem<1>::TOTAL);
+    cudaFuncSetAttribute(flash_fwd3_kernel<2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, Fwd3Smem<2>::TOTAL);
     configured = true;
   }
-  if (head_dim == 64) flash_fwd3_kernel<1><<<grid, FA_THREADS, Fwd3Smem<1>::TOTAL, st>>>(tq, tk, tv, p);
-  else flash_fwd3_kernel<2><<<grid, FA_THREADS, Fwd3Smem<2>::TOTAL, st>>>(tq, tk, tv, p);
+  const bool ext = p.gate || p.chunk;
+  if (head_dim == 64 && ext) flash_fwd3_kernel<1, true><<<grid, FA_THREADS, Fwd3Smem<1>::TOTAL, st>>>(tq, tk, tv, p);
+  else if (head_dim == 64) flash_fwd3_kernel<1, false><<<grid, FA_THREADS, Fwd3Smem<1>::TOTAL, st>>>(tq, tk, tv, p);
+  else if (ext) flash_fwd3_kernel<2, true><<<grid, FA_THREADS, Fwd3Smem<2>::TOTAL, st>>>(tq, tk, tv, p);
+  else flash_fwd3_kernel<2, false><<<grid, FA_THREADS, Fwd3Smem<2>::TOTAL, st>>>(tq, tk, tv, p);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
 }

@@ -87,12 +87,13 @@ constexpr int KV_MAX_PAIRS = 512;
 template <typename TI, typename TC, int NCH>
 __global__ void __launch_bounds__(512) qkv_prep_kernel(const QkvPrep p) {
   __shared__ float red[2][16];
-  __shared__ float2 turn[KV_MAX_PAIRS];
+  __shared__ __align__(16) float2 turn[KV_MAX_PAIRS];
   const int tid = threadIdx.x, nt = blockDim.x;
   const size_t t = blockIdx.x;
   const TI* row = static_cast<const TI*>(p.in) + t * p.in_ld;
   const int per = p.Dp / 8, nq = p.H * per, n = (p.H + p.G) * per;
   const int pos = p.tok_pos[t];
+  const int page = p.page_table[(size_t)p.rows[p.tok_seq[t]] * p.max_pages + pos / KV_PAGE];
   auto source = [&](int c) { return c < nq ? row + p.off_q + c * 8 : row + p.off_k + (c - nq) * 8; };
   Eight<TI> keep[NCH > 0 ? NCH : 1];
   float sq = 0.f, sk = 0.f;
@@ -109,9 +110,9 @@ __global__ void __launch_bounds__(512) qkv_prep_kernel(const QkvPrep p) {
     for (int i = 0; i < (NCH > 0 ? NCH : 1); ++i)
       if (tid + i * nt < n) keep[i].load(source(tid + i * nt));
   }
-  for (int i = tid; i < p.pairs; i += nt) {
-    float s, c;
-    sincosf((float)pos * p.freq[i], &s, &c);
+  for (int i = tid; i < (p.pairs + 3) / 4 * 4; i += nt) {
+    float s = 0.f, c = 1.f;
+    if (i < p.pairs) sincosf((float)pos * p.freq[i], &s, &c);
     turn[i] = make_float2(c, s);
   }
   if (NCH > 0) {
@@ -138,16 +139,17 @@ __global__ void __launch_bounds__(512) qkv_prep_kernel(const QkvPrep p) {
   }
   const float rq = p.q_norm ? 1.0f / sqrtf(sq / (float)(p.H * p.D) + p.eps) : 1.0f;
   const float rk = p.k_norm ? 1.0f / sqrtf(sk / (float)(p.G * p.D) + p.eps) : 1.0f;
-  const int page = p.page_table[(size_t)p.rows[p.tok_seq[t]] * p.max_pages + pos / KV_PAGE];
   TC* pool = static_cast<TC*>(p.pool) + (size_t)page * p.G * 2 * KV_PAGE * p.Dp + (size_t)(pos % KV_PAGE) * p.Dp;
+  const float inv_per = 1.0f / (float)per;
   auto write = [&](const Eight<TI>& e, int c) {
     const bool is_q = c < nq;
-    const int kc = c - nq, col = (is_q ? c : kc) * 8, d0 = col % p.Dp;
+    const int piece = is_q ? c : c - nq, col = piece * 8;
+    const int head = (int)(((float)piece + 0.5f) * inv_per), d0 = (piece - head * per) * 8;  // far below the fp32 range of exact integers
+    TC* slot = pool + (size_t)head * (2 * KV_PAGE) * p.Dp + d0;                                // (key heads)
     float f[8];
     e.get(f);
     Eight<TC> o;
     if (!is_q) {  // the value: as projected
-      TC* dst = pool + (size_t)((kc / per) * 2 + 1) * KV_PAGE * p.Dp + d0;
       if (p.off_v == p.off_k) {
         o.set(f);
       } else {
@@ -157,7 +159,7 @@ __global__ void __launch_bounds__(512) qkv_prep_kernel(const QkvPrep p) {
         ve.get(v);
         o.set(v);
       }
-      o.store(dst);
+      o.store(slot + KV_PAGE * p.Dp);
     }
     const float* w = is_q ? p.q_norm : p.k_norm;
     if (w) {
@@ -169,19 +171,23 @@ __global__ void __launch_bounds__(512) qkv_prep_kernel(const QkvPrep p) {
 #pragma unroll
       for (int i = 0; i < 8; ++i) f[i] = f[i] * r * wv[i];
     }
+    if (d0 < 2 * p.pairs) {
+      // entries past the last pair turn by nothing
+      const float4* tp = reinterpret_cast<const float4*>(turn + d0 / 2);
+      const float4 ta = tp[0], tb = tp[1];
+      const float tc[4] = {ta.x, ta.z, tb.x, tb.z}, ts[4] = {ta.y, ta.w, tb.y, tb.w};
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
-      if (d0 / 2 + i < p.pairs) {
-        const float2 cs = turn[d0 / 2 + i];
+      for (int i = 0; i < 4; ++i) {
         const float u = f[2 * i], v = f[2 * i + 1];
-        f[2 * i] = u * cs.x - v * cs.y;
-        f[2 * i + 1] = v * cs.x + u * cs.y;
+        f[2 * i] = u * tc[i] - v * ts[i];
+        f[2 * i + 1] = v * tc[i] + u * ts[i];
       }
+    }
     o.set(f);
     if (is_q) {
       o.store(static_cast<TC*>(p.q_out) + t * (size_t)(p.H * p.Dp) + col);
     } else {
-      o.store(pool + (size_t)(kc / per) * 2 * KV_PAGE * p.Dp + d0);
+      o.store(slot);
       if (p.k_out) o.store(static_cast<TC*>(p.k_out) + t * (size_t)(p.G * p.Dp) + col);
     }
   };

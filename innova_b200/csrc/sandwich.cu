@@ -157,9 +157,10 @@ __global__ void __launch_bounds__(512) sandwich_any_kernel(const SandwichParams 
 
 template <typename YT, typename HT>
 static int sandwich_launch(const SandwichParams& p, int n, bool vec, cudaStream_t st) {
-  const int cap = n <= 148 ? 512 : 256;  // few rows: one short pass over a row
-  const int e4 = p.E / 4, rounds = (e4 + cap - 1) / cap;
-  const int threads = ((e4 + (rounds > 0 ? rounds : 1) - 1) / (rounds > 0 ? rounds : 1) + 31) / 32 * 32;
+  // few rows: one short pass over a row, its latency is all there is; many: enough values per thread to pay for the two block sums
+  const int e4 = p.E / 4, few = (e4 + 511) / 512;
+  const int want = n <= 148 || e4 < 256 ? 1 : e4 < 512 ? 2 : 4, rounds = few > want ? few : want;
+  const int threads = ((e4 + rounds - 1) / rounds + 31) / 32 * 32;
   if (!vec || rounds > 12) sandwich_any_kernel<YT, HT><<<n, 256, 0, st>>>(p);
   else if (rounds <= 1) sandwich_kernel<YT, HT, 1><<<n, threads, 0, st>>>(p);
   else if (rounds <= 2) sandwich_kernel<YT, HT, 2><<<n, threads, 0, st>>>(p);

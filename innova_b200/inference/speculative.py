@@ -133,6 +133,9 @@ class SpeculativeDecoder:
         self.gen = torch.Generator().manual_seed(seed)
         self.stats = RejectionStats()
         self.acc_ema = 0.5
+        for g in (target, draft):
+            if hasattr(g.cache, "rewind"):               # a cache that gives pages back early keeps what rejected drafts lead back to
+                g.cache.rewind = max_gamma + 2
 
     def adapt_gamma(self, round_rate: float):
         """gamma = round(5 * min(ema/(1-ema), 5)) clamped, as the reference adapts it."""

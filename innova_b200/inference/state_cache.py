@@ -13,6 +13,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import List, Optional, Sequence
 
+import numpy as np
 import torch
 
 from ..ops.delta_rule import CHUNK
@@ -48,8 +49,8 @@ class StepBatch:
             raise ValueError("a step needs at least one token per sequence")
         if len(set(rows)) != len(rows) or min(rows) < 0 or max(rows) >= cache.max_batch:
             raise ValueError(f"bad cache rows {list(rows)}")
-        flat = [int(t) for ts in tokens for t in ts]
-        if vocab is not None and not (0 <= min(flat) and max(flat) < vocab):
+        flat = np.concatenate([np.asarray(t, dtype=np.int64) for t in tokens])
+        if vocab is not None and not (0 <= flat.min() and flat.max() < vocab):
             raise ValueError(f"token id outside the vocabulary of {vocab}")
         self.n, self.T, self.max_len = len(lens), len(flat), max(lens)
         self.host_rows, self.host_start, self.lens = list(rows), [int(s) for s in start], lens
@@ -57,39 +58,36 @@ class StepBatch:
         self.single = self.max_len == 1              # one token per sequence: the decode kernels
         self.fresh = not any(self.host_start)        # whole prompts: nothing is read from the cache
         self.device = cache.device
-        cu = [0]
-        for n in lens:
-            cu.append(cu[-1] + n)
-        if want is None:
-            want = [c - 1 for c in cu[1:]]
+        want = np.cumsum(lens) - 1 if want is None else np.asarray(want, dtype=np.int64)
         self.n_want = len(want)
-        self.want_all = list(want) == list(range(self.T))
+        self.want_all = self.n_want == self.T and bool((want == np.arange(self.T)).all())
         self.n_chunks = sum(-(-n // CHUNK) for n in lens)      # the delta rule advances chunk by chunk inside a portion
         self._buf = torch.empty(5 * self.n + 2 + 3 * self.T + self.n_chunks + self.n_want, dtype=torch.int32, device=self.device)
         self._views()
-        self._fill(cache, flat, cu, want)
+        self._fill(cache, flat, want)
 
     def _views(self):
         sizes = [self.n, self.n, self.n, self.n + 1, self.n + 1, self.n_chunks, self.T, self.T, self.T, self.n_want]
         (self.start, self.rows, self.slots, self.cu, self.cu_chunk, self.chunk_seq, self.ids, self.tok_seq, self.tok_pos,
          self.want) = torch.split(self._buf[:sum(sizes)], sizes)
 
-    def _fill(self, cache, flat, cu, want):
-        seq = [i for i, n in enumerate(self.lens) for _ in range(n)]
-        pos = [s + k for s, n in zip(self.host_start, self.lens) for k in range(n)]
-        slots = [cache.slot_of(r) for r in self.host_rows]
-        cu_chunk = [0]
-        for n in self.lens:
-            cu_chunk.append(cu_chunk[-1] - (-n // CHUNK))
-        chunk_seq = [i for i, n in enumerate(self.lens) for _ in range(-(-n // CHUNK))]
-        host = torch.tensor(self.host_start + self.host_rows + slots + cu + cu_chunk + chunk_seq + flat + seq + pos + list(want), dtype=torch.int32)
-        self._buf[: host.numel()].copy_(host)
+    def _fill(self, cache, flat, want):
+        lens, start = np.asarray(self.lens), np.asarray(self.host_start)
+        seqs, chunks = np.arange(self.n), -(-lens // CHUNK)
+        ends = lambda n: np.concatenate(([0], np.cumsum(n)))
+        cu = ends(lens)
+        seq = np.repeat(seqs, lens)
+        parts = (start, self.host_rows, [cache.slot_of(r) for r in self.host_rows], cu, ends(chunks), np.repeat(seqs, chunks), flat, seq,
+                 start[seq] + np.arange(self.T) - cu[seq], want)
+        host = torch.empty(self._buf.numel(), dtype=torch.int32, pin_memory=self.device.type == "cuda")
+        np.concatenate(parts, out=host.numpy(), casting="unsafe")
+        self._buf.copy_(host, non_blocking=True)
 
     def refill(self, cache, tokens: Sequence[int], start: Sequence[int], rows: Sequence[int]):
         """Same shape, next step (one token per sequence): new values in the same device memory (a captured graph reads it)."""
         self.host_rows, self.host_start = list(rows), [int(s) for s in start]
         self.max_pos = max(self.host_start) + 1
-        self._fill(cache, [int(t) for t in tokens], list(range(self.n + 1)), range(self.n))
+        self._fill(cache, np.asarray(tokens), np.arange(self.n))
 
 
 class StepCache(PagedRows):

@@ -118,7 +118,7 @@ class GatedAttention(Mixer):
 
     @classmethod
     def check(cls, m: dict, layer: int):
-        if m["vdim"] != m["dim"]:
+        if m.get("vdim", m["dim"]) != m["dim"]:
             raise ValueError(f"layer {layer}: values are the keys, but vdim {m['vdim']} is not dim {m['dim']}")
         if m["heads"] % m["kv_heads"]:
             raise ValueError(f"layer {layer}: {m['heads']} heads do not share {m['kv_heads']} key heads evenly")

@@ -81,11 +81,16 @@ def first_visible(pos: int, window: Optional[int], chunk: Optional[int]) -> int:
 
 
 def cluster_shape(rows: int, groups: int, span: int):
-    """(CTAs, warps per CTA) that share one (row, key head): enough of them to fill the GPU, at least two pages per warp."""
-    pages, splits = -(-span // PAGE), 1
-    while splits < 8 and rows * groups * splits < 2 * 148 and pages >= 16 * splits:
-        splits *= 2
-    return splits, (8 if splits == 8 and rows * groups * splits <= 148 and pages >= 128 else 4)
+    """(CTAs, warps per CTA) that share one (row, key head): about 1024 warps in flight altogether, at least two pages each."""
+    pages, units = -(-span // PAGE), rows * groups
+    if 444 < units <= 888 and pages >= 128:
+        return 2, 4                  # one CTA per unit would leave the second wave of CTAs nearly empty
+    warps = 4
+    while warps < 32 and units * warps * 2 <= 1024 and pages >= warps * 4:
+        warps *= 2
+    if warps == 32 and units <= 8 and pages >= 256:
+        return 8, 8
+    return {4: (1, 4), 8: (1, 8), 16: (4, 4), 32: (8, 4)}[warps]
 
 
 def kv_attend(q: torch.Tensor, pool, page_table, heads: int, scale: float, batch, window: Optional[int] = None, chunk: Optional[int] = None,
