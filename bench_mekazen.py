@@ -106,6 +106,7 @@ def kernel_section(size="2k"):
     from innova_b200.inference.state_cache import KeyValues, StepBatch, StepCache
     from innova_b200.ops import kv_attention as ka
     from innova_b200.ops import latent_attention as la
+    from innova_b200.ops.hyper import gated_silu
     from innova_b200.ops.sandwich import sandwich_step, softcap_
     E, F, H, G, V = SIZES[size]
     D = 128
@@ -180,8 +181,12 @@ def kernel_section(size="2k"):
                    cold(lambda: la.packed_flash(q, k, v, H, D, 0.09, None, b, kv_heads=G, chunk=chunk, gate=gate)), tflop=fl(chunk))
         with torch.no_grad():
             report("flash_attention", f"{B} x {S} H{H} G{G} D{D}", cold(lambda: ops.flash_attention(qkv, H, G, D)), tflop=fl(S), like="packed_flash")
+            short = qkv.view(T // 1024, 1024, -1)        # the same work as chunks of 1024
+            report("flash_attention", f"{T // 1024} x 1024 H{H} G{G} D{D}", cold(lambda: ops.flash_attention(short, H, G, D)), tflop=fl(1024), like="packed_flash")
     z = rand(512, V)
     report("softcap", f"512 x {V}", cold(lambda: softcap_(z, 30.0)), z.numel() * 8 / 1e9)
+    gu = rand(8192, 2 * F).to(bf)
+    report("gated_silu", f"8192 x {F}", cold(lambda: gated_silu(gu, F, bf)), gu.numel() * 3 / 1e9, like="softcap")
 
 
 def main(section="all", sizes=None):

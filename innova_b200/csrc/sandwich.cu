@@ -171,10 +171,19 @@ static int sandwich_launch(const SandwichParams& p, int n, bool vec, cudaStream_
   return e == cudaSuccess ? 0 : -(int)e;
 }
 
-// x <- cap * tanh(x / cap), rows of `cols` values `ld` apart
-__global__ void __launch_bounds__(256) softcap_kernel(float* x, int ld, int cols, float cap) {
+// x <- cap * tanh(x / cap), rows of `cols` values `ld` apart; V values per access
+template <int V>
+__global__ void __launch_bounds__(256) softcap_kernel(float* x, int ld, int cols, float cap, float inv_cap) {
   float* r = x + (size_t)blockIdx.x * ld;
-  for (int c = blockIdx.y * 256 + threadIdx.x; c < cols; c += gridDim.y * 256) r[c] = cap * tanhf(r[c] / cap);
+  for (int c = (blockIdx.y * 256 + threadIdx.x) * V; c < cols; c += gridDim.y * 256 * V) {
+    if (V == 4 && c + 4 <= cols) {
+      float4 v = *reinterpret_cast<float4*>(r + c);
+      v.x = cap * tanhf(v.x * inv_cap); v.y = cap * tanhf(v.y * inv_cap); v.z = cap * tanhf(v.z * inv_cap); v.w = cap * tanhf(v.w * inv_cap);
+      *reinterpret_cast<float4*>(r + c) = v;
+    } else {
+      for (int i = c; i < min(c + V, cols); ++i) r[i] = cap * tanhf(r[i] * inv_cap);
+    }
+  }
 }
 
 }  // namespace inv
@@ -198,9 +207,11 @@ extern "C" int inv_sandwich_step(float* x, const int* ids, const void* table, in
 extern "C" int inv_softcap(float* x, int ld, int rows, int cols, float cap, void* stream) {
   if (!(cap > 0.f)) return -ERR_BAD_ARG;
   if (rows <= 0 || cols <= 0) return 0;
-  int by = (cols + 255) / 256;
-  if (rows > 148 * 8 && by > 16) by = 16;
-  softcap_kernel<<<dim3(rows, by), 256, 0, (cudaStream_t)stream>>>(x, ld, cols, cap);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (ld % 4 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0)
+    softcap_kernel<4><<<dim3(rows, (cols + 2047) / 2048), 256, 0, st>>>(x, ld, cols, cap, 1.0f / cap);
+  else
+    softcap_kernel<1><<<dim3(rows, (cols + 1023) / 1024), 256, 0, st>>>(x, ld, cols, cap, 1.0f / cap);
   const cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
 }

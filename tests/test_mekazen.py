@@ -104,9 +104,12 @@ def test_fp32_output_of_small_products_enters_a_bf16_model(dev):
 
 @pytest.mark.parametrize("rows", [3, 50])
 def test_softcap(dev, rows):
-    z = torch.randn(rows, 300) * 40
-    got = softcap_(z.clone().to(dev[0])[:, :297], 30.0).cpu()
-    assert torch.allclose(got, oracle.softcap(z[:, :297], 30.0), atol=1e-5) and got.abs().max() <= 30.0
+    for ld, n in ((300, 297), (301, 301), (5000, 4999)):
+        z = torch.randn(rows, ld) * 40
+        x = z.clone().to(dev[0])
+        got = softcap_(x[:, :n], 30.0).cpu()
+        assert torch.allclose(got, oracle.softcap(z[:, :n], 30.0), atol=1e-5) and got.abs().max() <= 30.0
+        assert torch.equal(x[:, n:].cpu(), z[:, n:])
 
 
 @pytest.mark.gpu
