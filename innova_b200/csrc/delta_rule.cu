@@ -114,7 +114,7 @@ __global__ void __launch_bounds__(CK_THREADS, 6) delta_chunk_kernel(const T* __r
 #pragma unroll
       for (int k = 0; k < TAPS - 1; ++k) {
         const int t = tb + k - (TAPS - 1);
-        in[k] = TAPS - 1 - k < s.taps ? conv_in(proj, ld, ring, s, row0, start, pos0 + t, c) : 0.f;
+        in[k] = TAPS - 1 - k < s.taps && t < n ? conv_in(proj, ld, ring, s, row0, start, pos0 + t, c) : 0.f;  // (the second half of a short chunk has no rows)
       }
 #pragma unroll
       for (int k = 0; k < HALF; ++k) in[TAPS - 1 + k] = tb + k < n ? dr_ld(col + (long)(tb + k) * ld) : 0.f;
