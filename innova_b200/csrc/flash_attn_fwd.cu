@@ -267,11 +267,10 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       __syncwarp();
       if (lane == 0) mbar_arrive(p_full);
     }
-    const size_t grow = (p.cu ? (size_t)row_base : (size_t)b * S) + row;
     uint4 gv[EXT ? D / 8 : 1];                    // the row's gate, requested while the last PV MMA runs
     const bool gated = EXT && p.gate != nullptr;
     if (gated && row < S) {
-      const __nv_bfloat16* gate = p.gate + grow * p.ld_gate + h * D;
+      const __nv_bfloat16* gate = p.gate + ((p.cu ? (size_t)row_base : (size_t)b * S) + row) * p.ld_gate + h * D;
 #pragma unroll
       for (int i = 0; i < (EXT ? D / 8 : 1); ++i) gv[i] = *reinterpret_cast<const uint4*>(gate + i * 8);
     }
@@ -279,7 +278,7 @@ flash_fwd3_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     if (ok) {
       tc_fence_after();
       const float inv_l = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* dst = p.out + grow * p.ld_o + h * D;
+      __nv_bfloat16* dst = p.out + ((p.cu ? (size_t)row_base : (size_t)b * S) + row) * p.ld_o + h * D;
 #pragma unroll (EXT ? D / 32 : 1)
       for (int cc = 0; cc < D / 32; ++cc) {
         uint32_t rr[32];
